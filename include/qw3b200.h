@@ -304,6 +304,14 @@ int  qb_model_load_gguf(qb_ctx *ctx, const char *path, qb_model **out, qb_model_
 /* The parsing half alone (no device needed): configuration, number of F32 / Q8_0 tensors and their bytes. */
 int  qb_gguf_read_config(const char *path, qb_model_config *cfg_out, uint64_t *n_tensors_out, uint64_t *tensor_bytes_out);
 const qb_model_config *qb_model_get_config(const qb_model *m);
+/* A model by path: a GGUF file (qwen35), or a folder with config.json and model.safetensors whose config.json names an
+ * architecture of the loader table ("Kezilix": a layered model -- retention and latent-attention layers, dense
+ * feed-forwards, a looped span -- with bfloat16 weights).  f32 != 0: every product and activation in 32 bits (layered
+ * models only, QB_ERR_UNSUPPORTED otherwise).  cfg_out (may be NULL): of a layered model, only n_layers, n_embd,
+ * vocab_size and rms_eps are set. */
+int  qb_model_load(qb_ctx *ctx, const char *path, int f32, qb_model **out, qb_model_config *cfg_out);
+/* A layered model of the given configuration (the text of a config.json) with seeded random weights. */
+int  qb_model_create_layered_synth(qb_ctx *ctx, const char *config_json, uint64_t seed, int f32, qb_model **out);
 void qb_model_destroy(qb_ctx *ctx, qb_model *m);
 size_t qb_model_weight_bytes(const qb_model *m);
 
@@ -386,6 +394,9 @@ int qb_prefill(qb_ctx *ctx, qb_batch *b, uint32_t seq, const int32_t *tokens_hos
  * src/qwen_native_backend.cpp:4482-4530): K/V, recurrent state and MTP prefix advance; no LM head, no token is chosen,
  * nothing is counted as emitted or recorded as seen beyond the prompt tokens.  Finish with qb_prefill(_sampled). */
 int qb_prefill_chunk(qb_ctx *ctx, qb_batch *b, uint32_t seq, const int32_t *tokens_host, uint32_t n);
+/* qb_prefill_chunk that also scores: logits_host[i][vocab] = the logits at token want[i] (0-based in this part). */
+int qb_prefill_logits(qb_ctx *ctx, qb_batch *b, uint32_t seq, const int32_t *tokens_host, uint32_t n, const int32_t *want, uint32_t n_want,
+                      float *logits_host);
 /* Sampling parameters of a request (GenerationOptions, include/qw3/qw3.hpp:222-230). */
 typedef struct qb_sampling { float temp, top_p; int32_t top_k; float min_p; } qb_sampling;
 /* The end of a sampled request's prompt: as qb_prefill, but the first token is drawn from the last row's logits with
@@ -396,6 +407,10 @@ int qb_prefill_sampled(qb_ctx *ctx, qb_batch *b, uint32_t seq, const int32_t *to
 /* forward_one_token + argmax (src/qwen_executor.cpp:5446-5816): one non-speculative greedy step
  * for every sequence.  Emits one token per sequence. */
 int qb_decode_greedy_step(qb_ctx *ctx, qb_batch *b);
+
+/* The same with sampling: sequence s draws its token with u_host[s] (pick_from_last_logits of a plain sampled step,
+ * src/qwen_native_backend.cpp:15399-15428; token penalties as qb_batch_set_penalties). */
+int qb_decode_sampled_step(qb_ctx *ctx, qb_batch *b, const qb_sampling *samp, const double *u_host);
 
 /* forward_mtp_draft_chain_with_prefix_device (src/qwen_executor.cpp:6942-7023): k chained MTP-head
  * forwards per sequence, argmax kept on the device. */
@@ -491,6 +506,10 @@ void qb_snapshot_free(qb_ctx *ctx, qb_snapshot *snap);
 int qb_debug_last_logits(qb_ctx *ctx, qb_batch *b, float *host_out, uint32_t max_rows, uint32_t *rows_out);
 /* Drafts of the last qb_mtp_draft / qb_mtp_force_drafts: int32 [n_seqs][k] (test aid, syncs). */
 int qb_debug_last_drafts(qb_ctx *ctx, qb_batch *b, int32_t *host_out);
+/* Residual rows of a layered model after every layer run of the last forward: while on, float [runs][rows][n_embd] (before
+ * what the loop adds in front of a pass).  host_out may be NULL to ask for the sizes. */
+int qb_debug_layer_trace(qb_ctx *ctx, qb_batch *b, int on);
+int qb_debug_layer_trace_read(qb_ctx *ctx, qb_batch *b, float *host_out, uint32_t max_rows, uint32_t *runs_out, uint32_t *rows_out);
 /* Per-launch CUDA-event timing of the Q8 GEMM kernels on the context stream (the reference's
  * per-op timing, src/qwen_executor.cpp:1788-1804, without its synchronise-per-op): enable, run,
  * then read the summed duration, the summed algorithmic bytes and the number of launches. */

@@ -3,6 +3,7 @@
 The library is CUDA-only: loading works anywhere, but creating a context without a B200 raises.
 """
 import ctypes as C
+import json
 import os
 
 import numpy as np
@@ -96,6 +97,8 @@ SIGNATURES = {
     "qb_model_create_synth": (i32, [vp, C.POINTER(ModelConfig), u64, C.POINTER(vp)]),
     "qb_model_create": (i32, [vp, C.POINTER(ModelConfig), C.POINTER(TensorDesc), sz, C.POINTER(vp)]),
     "qb_model_load_gguf": (i32, [vp, C.c_char_p, C.POINTER(vp), C.POINTER(ModelConfig)]),
+    "qb_model_load": (i32, [vp, C.c_char_p, i32, C.POINTER(vp), C.POINTER(ModelConfig)]),
+    "qb_model_create_layered_synth": (i32, [vp, C.c_char_p, u64, i32, C.POINTER(vp)]),
     "qb_gguf_read_config": (i32, [C.c_char_p, C.POINTER(ModelConfig), C.POINTER(u64), C.POINTER(u64)]),
     "qb_tokenizer_load_gguf": (i32, [C.c_char_p, C.POINTER(vp)]),
     "qb_tokenizer_create": (i32, [C.POINTER(C.c_char_p), C.POINTER(u32), u32, C.POINTER(C.c_char_p), C.POINTER(u32), u32, C.c_int32, C.c_int32, i32,
@@ -129,6 +132,8 @@ SIGNATURES = {
     "qb_batch_destroy": (None, [vp, vp]),
     "qb_prefill": (i32, [vp, vp, u32, vp, u32]),
     "qb_prefill_chunk": (i32, [vp, vp, u32, vp, u32]),
+    "qb_prefill_logits": (i32, [vp, vp, u32, vp, u32, vp, u32, vp]),
+    "qb_decode_sampled_step": (i32, [vp, vp, C.POINTER(Sampling), vp]),
     "qb_prefill_sampled": (i32, [vp, vp, u32, vp, u32, C.POINTER(Sampling), C.c_double]),
     "qb_decode_greedy_step": (i32, [vp, vp]),
     "qb_mtp_draft": (i32, [vp, vp]),
@@ -154,6 +159,8 @@ SIGNATURES = {
     "qb_snapshot_free": (None, [vp, vp]),
     "qb_debug_last_logits": (i32, [vp, vp, vp, u32, C.POINTER(u32)]),
     "qb_debug_last_drafts": (i32, [vp, vp, vp]),
+    "qb_debug_layer_trace": (i32, [vp, vp, i32]),
+    "qb_debug_layer_trace_read": (i32, [vp, vp, vp, u32, C.POINTER(u32), C.POINTER(u32)]),
     "qb_prof_enable": (i32, [vp, i32]),
     "qb_prof_summary": (i32, [vp, C.POINTER(C.c_double), C.POINTER(C.c_double), C.POINTER(C.c_int64)]),
     "qb_trace_enable": (i32, [vp, i32]),
@@ -179,6 +186,10 @@ class QbError(RuntimeError):
     pass
 
 
+class QbUnsupported(QbError):
+    """The library has no form of what was asked for (QB_ERR_UNSUPPORTED)."""
+
+
 def lib():
     """Loads the CUDA library; raises if it has not been built (there is no CPU fallback)."""
     global _LIB
@@ -196,7 +207,7 @@ def lib():
 
 def check(status):
     if status != 0:
-        raise QbError("qw3b200 error %d: %s" % (status, lib().qb_last_error().decode()))
+        raise (QbUnsupported if status == 3 else QbError)("qw3b200 error %d: %s" % (status, lib().qb_last_error().decode()))
 
 
 def _np_ptr(a):
@@ -573,6 +584,27 @@ class Model:
         self.h, self.cfg = h, cfg
         return self
 
+    @classmethod
+    def load(cls, ctx, path, dtype="bfloat16"):
+        """A GGUF file, or a model folder (config.json, model.safetensors) of an architecture the library knows.
+        dtype float32: every product and activation in 32 bits, where the family has that form."""
+        self = cls.__new__(cls)
+        self.ctx = ctx
+        h, cfg = vp(), ModelConfig()
+        check(lib().qb_model_load(ctx.h, os.fsencode(path), int(dtype == "float32"), C.byref(h), C.byref(cfg)))
+        self.h, self.cfg = h, cfg
+        return self
+
+    @classmethod
+    def layered_synth(cls, ctx, config, seed, dtype="bfloat16"):
+        """A layered model with seeded random weights; config: the dict of a config.json."""
+        self = cls.__new__(cls)
+        self.ctx = ctx
+        h = vp()
+        check(lib().qb_model_create_layered_synth(ctx.h, json.dumps(config).encode(), seed, int(dtype == "float32"), C.byref(h)))
+        self.h, self.cfg = h, ModelConfig.from_buffer_copy(lib().qb_model_get_config(h).contents)
+        return self
+
     @property
     def weight_bytes(self):
         return int(lib().qb_model_weight_bytes(self.h))
@@ -635,6 +667,13 @@ class Batch:
         fn = lib().qb_prefill_chunk if more else lib().qb_prefill
         check(fn(self.ctx.h, self.h, seq, _np_ptr(t), len(t)))
 
+    def score(self, seq, tokens, want):
+        """prefill(..., more=True) that returns the logits [len(want)][vocab] at the places `want` among these tokens."""
+        t, w = np.ascontiguousarray(tokens, np.int32), np.ascontiguousarray(want, np.int32)
+        out = np.empty((len(w), self.model.cfg.vocab_size), np.float32)
+        check(lib().qb_prefill_logits(self.ctx.h, self.h, seq, _np_ptr(t), len(t), _np_ptr(w), len(w), _np_ptr(out)))
+        return out
+
     def prefill_sampled(self, seq, tokens, u, temp, top_p=1.0, top_k=0, min_p=0.0):
         """The end of a sampled request's prompt: the first token is drawn with the uniform draw u."""
         t = np.ascontiguousarray(tokens, np.int32)
@@ -643,6 +682,12 @@ class Batch:
 
     def greedy_step(self):
         check(lib().qb_decode_greedy_step(self.ctx.h, self.h))
+
+    def sampled_step(self, u, temp, top_p=1.0, top_k=0, min_p=0.0):
+        """A plain sampled step: sequence s draws with u[s]."""
+        u = np.ascontiguousarray(u, np.float64).reshape(-1)
+        sp = Sampling(temp, top_p, top_k, min_p)
+        check(lib().qb_decode_sampled_step(self.ctx.h, self.h, C.byref(sp), _np_ptr(u)))
 
     def mtp_draft(self):
         check(lib().qb_mtp_draft(self.ctx.h, self.h))
@@ -746,6 +791,17 @@ class Batch:
         p = C.c_int32()
         check(lib().qb_seq_position(self.ctx.h, self.h, seq, C.byref(p)))
         return p.value
+
+    def layer_trace(self, on=True):
+        check(lib().qb_debug_layer_trace(self.ctx.h, self.h, 1 if on else 0))
+
+    def layer_trace_read(self):
+        """Residual rows of the last forward after every layer run: float32 [runs][rows][n_embd]."""
+        r, n = u32(), u32()
+        check(lib().qb_debug_layer_trace_read(self.ctx.h, self.h, None, 1 << 20, C.byref(r), C.byref(n)))
+        out = np.empty((r.value, n.value, self.model.cfg.n_embd), np.float32)
+        check(lib().qb_debug_layer_trace_read(self.ctx.h, self.h, _np_ptr(out), n.value, C.byref(r), C.byref(n)))
+        return out
 
     def last_drafts(self):
         out = np.zeros((self.n_seqs, self.k), np.int32)

@@ -10,10 +10,13 @@
 // All per-step control values (positions, selected state slot, current token, drafts) live in
 // device memory and are updated by kernels, so a step needs no host decision and no mid-step
 // synchronisation; the host reads back one small record per step.
-#include "qb_internal.h"
-#include "page_pool.h"
+#include "engine.h"
+#include "json_reader.h"
 
+#include <fstream>
+#include <sstream>
 #include <string>
+#include <sys/stat.h>
 
 namespace {
 
@@ -27,45 +30,11 @@ inline double urand(uint64_t seed, uint32_t stream, uint64_t i) {
     return (double)(qs_rand_u32(seed, stream, i) >> 8) / 16777216.0;
 }
 
-struct LayerW {
-    bool recurrent = false;
-    qb_weight *w_in = nullptr;       // attention: [q(+gate) ; k ; v]   DeltaNet: [qkv ; z ; alpha ; beta]
-    qb_weight *w_out = nullptr;      // attn_output / ssm_out
-    qb_weight *w_gate_up = nullptr;  // [gate ; up]
-    qb_weight *w_down = nullptr;
-    qb_weight w_kv;                  // view of the k and v rows of w_in (attention layers)
-    float *conv_w = nullptr, *ssm_a = nullptr, *dt_bias = nullptr;
-    // RMSNorm gains (attn_norm, ffn_norm / post_attention_norm, attn_q_norm, attn_k_norm, ssm_norm)
-    const float *attn_norm = nullptr, *ffn_norm = nullptr, *q_norm = nullptr, *k_norm = nullptr, *ssm_norm = nullptr;
-};
-
 }  // namespace
-
-struct qb_model {
-    qb_model_config cfg;
-    std::vector<LayerW> layers;      // n_layers (+ the MTP layer last)
-    qb_weight *token_embd = nullptr, *output = nullptr, *eh_proj = nullptr;
-    // MTP head: embedding table and LM head (nextn.embed_tokens / nextn.shared_head_head, else the target's)
-    qb_weight *mtp_embd = nullptr, *mtp_head = nullptr;
-    bool output_tied = false;        // no output.weight: the LM head is token_embd
-    uint32_t tp_rank = 0, tp_world = 1;   // FFN weights are shard tp_rank of tp_world (tensor-parallel form), else whole
-    float *ones = nullptr;           // every RMSNorm gain of the seeded model is 1.0
-    const float *output_norm = nullptr, *enorm = nullptr, *hnorm = nullptr, *shared_head_norm = nullptr;
-    std::vector<float *> owned_f32;  // fp32 tensors uploaded for this model
-    float *inv_freq = nullptr;
-    size_t weight_bytes = 0;
-    uint32_t inner() const { return cfg.n_heads * cfg.head_dim; }
-    uint32_t kvd() const { return cfg.n_kv_heads * cfg.head_dim; }
-    uint32_t attn_in() const { return 2 * inner() + 2 * kvd(); }
-    uint32_t qkv_dim() const { return (2 * cfg.ssm_num_k_heads + cfg.ssm_num_v_heads) * cfg.ssm_head_dim; }
-    uint32_t vdim() const { return cfg.ssm_num_v_heads * cfg.ssm_head_dim; }
-    uint32_t dn_in() const { return qkv_dim() + vdim() + 2 * cfg.ssm_num_v_heads; }
-    bool is_attn(uint32_t i) const { return cfg.full_attention_interval && ((i + 1) % cfg.full_attention_interval) == 0; }
-};
 
 static size_t weight_bytes_of(const qb_weight *w) { return (size_t)w->rows * w->cols / 32 * 34; }
 
-static int upload_f32(qb_ctx *ctx, const std::vector<float> &v, float **out) {
+int qb_upload_f32(qb_ctx *ctx, const std::vector<float> &v, float **out) {
     QB_CUDA(cudaMalloc(out, v.size() * sizeof(float)));
     QB_CUDA(cudaMemcpyAsync(*out, v.data(), v.size() * sizeof(float), cudaMemcpyHostToDevice, ctx->stream));
     QB_CUDA(cudaStreamSynchronize(ctx->stream));
@@ -102,9 +71,9 @@ static int build_layer(qb_ctx *ctx, qb_model *m, LayerW &L, uint32_t il, bool re
             sa[v] = (float)(-std::exp(urand(seed, tensor_id(il, T_SSM_A), v) * std::log(16.0)));
             dt[v] = (float)(-4.0 + 3.0 * urand(seed, tensor_id(il, T_SSM_DT), v));
         }
-        QB_TRY(upload_f32(ctx, conv, &L.conv_w));
-        QB_TRY(upload_f32(ctx, sa, &L.ssm_a));
-        QB_TRY(upload_f32(ctx, dt, &L.dt_bias));
+        QB_TRY(qb_upload_f32(ctx, conv, &L.conv_w));
+        QB_TRY(qb_upload_f32(ctx, sa, &L.ssm_a));
+        QB_TRY(qb_upload_f32(ctx, dt, &L.dt_bias));
     }
     // gate and up interleaved in groups of 64 rows: a 128-row tile holds both halves of 64 hidden indices.  In the
     // tensor-parallel form this rank holds FFN indices [lo, lo + f): those rows of gate and up, those columns of down.
@@ -121,6 +90,7 @@ static int build_layer(qb_ctx *ctx, qb_model *m, LayerW &L, uint32_t il, bool re
 }
 
 extern "C" void qb_model_destroy(qb_ctx *ctx, qb_model *m);
+extern const QbArch ARCH_QWEN35;
 
 // Shape checks shared by every model constructor, the all-ones gain vector and the RoPE frequencies.
 static int model_begin(qb_ctx *ctx, const qb_model_config &c, qb_model **out) {
@@ -136,12 +106,13 @@ static int model_begin(qb_ctx *ctx, const qb_model_config &c, qb_model **out) {
     QB_CUDA(cudaSetDevice(ctx->device));
     qb_model *m = new qb_model();
     m->cfg = c;
+    m->arch = &ARCH_QWEN35;
     *out = m;
     std::vector<float> ones(std::max({c.n_embd, c.head_dim, c.ssm_head_dim}), 1.0f);
-    QB_TRY(upload_f32(ctx, ones, &m->ones));
+    QB_TRY(qb_upload_f32(ctx, ones, &m->ones));
     std::vector<float> invf(c.rope_dim / 2);
     for (uint32_t i = 0; i < c.rope_dim / 2; ++i) invf[i] = (float)std::pow((double)c.rope_theta, -2.0 * (double)i / (double)c.rope_dim);
-    QB_TRY(upload_f32(ctx, invf, &m->inv_freq));
+    QB_TRY(qb_upload_f32(ctx, invf, &m->inv_freq));
     m->layers.resize(c.n_layers + (c.mtp_layers ? 1 : 0));
     return QB_OK;
 }
@@ -352,6 +323,11 @@ extern "C" const qb_model_config *qb_model_get_config(const qb_model *m) { retur
 extern "C" void qb_model_destroy(qb_ctx *ctx, qb_model *m) {
     if (!m) return;
     cudaStreamSynchronize(ctx->stream);
+    if (m->arch) m->arch->model_free(ctx, m);
+    for (float *p : m->owned_f32) cudaFree(p);
+    delete m;
+}
+static void qwen35_model_free(qb_ctx *ctx, qb_model *m) {
     std::vector<const float *> owned(m->owned_f32.begin(), m->owned_f32.end());
     auto is_owned = [&](const float *p) { return std::find(owned.begin(), owned.end(), p) != owned.end(); };
     for (LayerW &L : m->layers) {
@@ -365,83 +341,14 @@ extern "C" void qb_model_destroy(qb_ctx *ctx, qb_model *m) {
     if (m->mtp_head && m->mtp_head != m->output) qb_weight_free(ctx, m->mtp_head);
     if (!m->output_tied) qb_weight_free(ctx, m->output);
     qb_weight_free(ctx, m->token_embd); qb_weight_free(ctx, m->eh_proj);
-    for (float *p : m->owned_f32) cudaFree(p);
     if (m->ones) cudaFree(m->ones);
     if (m->inv_freq) cudaFree(m->inv_freq);
-    delete m;
 }
 extern "C" size_t qb_model_weight_bytes(const qb_model *m) { return m->weight_bytes; }
 
 // ================================================================================================
 // sequences
 // ================================================================================================
-struct QBuf {   // quantised activation buffer for one K
-    int8_t *q = nullptr; float *d = nullptr; uint32_t K = 0;
-};
-
-struct qb_batch {
-    qb_model *m = nullptr;
-    uint32_t n_seqs = 0, max_ctx = 0, k = 0, page_size = 0, pages_per_seq = 0, rows_cap = 0, chunk = 0, logit_rows = 0;
-    bool attn_tc = false;                  // decode / verify attention on the tensor-memory kernel: decided once, from n_seqs * max_ctx
-    uint32_t attn_split = 0;               // keys per attention split of this batch (absolute boundaries): decided once with attn_tc
-    uint32_t n_active = 0;                 // the decode steps run sequences [0, n_active); the rest keep their state untouched
-    std::vector<__half *> kc, vc;          // per layer (attention layers only), + MTP layer at index n_layers
-    std::vector<float *> state, conv;      // per layer (recurrent layers only): [n_seqs][k+1][...]
-    std::vector<float *> conv_alt;         // second conv-state buffer: a forward reads one and writes the other
-    int conv_par = 0;                      // which of the two holds the valid conv state (the same for all sequences)
-    int32_t *page_table = nullptr;         // [n_seqs][pages_per_seq]
-    // pooled form (qb_batch_create_pooled): the caches hold pool->total() pages shared by all sequences; a sequence's
-    // page-table row grows as its position grows and goes back to the pool at qb_seq_reset
-    QbPagePool *pool = nullptr;
-    std::vector<std::vector<int32_t>> seq_pages;   // host mirror of the page-table rows (pooled form)
-    std::vector<int32_t> chunk_end_pos;            // position after the sequence's last qb_prefill_chunk, -1 once anything else moved it
-    // device control block (all int32)
-    int32_t *ctl = nullptr;
-    int32_t *pos = nullptr, *sel = nullptr, *cur = nullptr, *drafts = nullptr, *zero_sel = nullptr;
-    int32_t *tok_buf = nullptr, *seqpos_buf = nullptr, *prefix_pos = nullptr, *prefix_tok = nullptr;
-    int32_t *out_rec = nullptr;            // [n_out (n_seqs) | tokens (n_seqs*(k+1)) | pos (n_seqs)]
-    int32_t *map_prevh = nullptr, *map_prefix = nullptr, *map_chunk = nullptr, *map_last = nullptr;
-    long long *stats = nullptr;            // [QB_STATS]: steps, drafted, accepted, emitted, rejecting steps, -, -, -, then steps by accepted length
-    int32_t *out_rec_host = nullptr;       // pinned mirror of out_rec
-    // activations
-    float *hid = nullptr;                  // [rows_cap + n_seqs][H]; rows rows_cap+s hold prev hidden of seq s
-    float *mtp_h = nullptr, *embd = nullptr, *act = nullptr, *parts = nullptr;
-    float *logits = nullptr, *am_val = nullptr, *att_acc = nullptr, *att_ml = nullptr;
-    int32_t *am_idx = nullptr;
-    QBuf xq_h, xq_attn, xq_dn, xq_ffn, xq_cat;
-    size_t parts_floats = 0;
-    std::vector<int32_t> host_pos;         // upper bound of pos per sequence
-    uint32_t last_logit_rows = 0;
-    int gemm_impl = 0;
-    double *samp_u = nullptr;              // [2][logit_rows]: acceptance draws, then residual draws (sampling mode)
-    uint32_t *seen = nullptr;              // [n_seqs][seen_words] bitmap of prompt + emitted tokens (token penalties), or null
-    uint32_t seen_words = 0;
-    float pen_presence = 0.0f, pen_repetition = 1.0f;
-    qb_tp_group *tp = nullptr;             // tensor-parallel FFN group of the batch's model shard, or null
-    float *normed = nullptr, *tp_y = nullptr;   // [rows_cap][H]: fp32 FFN input / all-reduced FFN output of the tensor-parallel form
-    int32_t *tok_stage = nullptr;          // pinned staging of the prompt tokens being ingested
-    int32_t *tok_all = nullptr;            // the same on the device: one copy per call, the chunks index into it
-    cudaEvent_t tok_ev = nullptr;          // that copy has landed (the staging area may be rewritten)
-    uint32_t tok_stage_cap = 0;
-    double *first_draw_stage = nullptr;    // pinned: the first-token draw of a sampled request per sequence
-    int32_t *limit = nullptr;              // [n_seqs] device: draft depth of the next step per sequence (<= k)
-    int32_t *limit_host = nullptr;         // pinned staging of the same
-    int32_t eos_token = -1;                // a draft equal to it ends the chain (-1: none)
-    void *swap_tmp = nullptr;              // one sequence's largest per-layer state block (qb_seq_swap)
-    size_t swap_bytes = 0;
-    // sampled steps: pinned staging ring of the step's draws (a slot is reused when its copy of four steps ago has landed)
-    static constexpr int SAMP_RING = 4;
-    double *samp_stage = nullptr;
-    cudaEvent_t samp_ev[SAMP_RING] = {};
-    uint32_t samp_slot = 0;
-    // position probe: keeps host_pos near the device's positions when nobody reads the step records (see probe_tick)
-    int32_t *probe_host = nullptr;         // pinned [n_seqs]
-    cudaEvent_t probe_ev = nullptr;
-    bool probe_pending = false;
-    int32_t probe_adv = 0;                 // positions enqueued since the probe's copy
-    uint32_t steps_since_probe = 0;
-};
-
 static size_t ctl_count(const qb_batch *b);
 static constexpr size_t QB_STATS = 16;
 
@@ -452,38 +359,29 @@ static int alloc_qbuf(QBuf &b, uint32_t rows, uint32_t K) {
     return QB_OK;
 }
 
-static uint32_t env_u32(const char *name, uint32_t dflt) {
+uint32_t qb_env_u32(const char *name, uint32_t dflt) {
     const char *v = getenv(name);
     return (v && *v) ? (uint32_t)strtoul(v, nullptr, 10) : dflt;
 }
 
-static int batch_create(qb_ctx *ctx, qb_model *m, uint32_t n_seqs, uint32_t max_ctx, uint32_t draft_k,
-                        uint32_t page_size, int page_order, uint32_t pool_pages, qb_batch **out) {
-    QB_REQUIRE(ctx && m && out && n_seqs > 0 && max_ctx > 0 && page_size > 0, "qb_batch_create: bad arguments");
-    QB_REQUIRE(draft_k <= 7, "draft depth %u unsupported (<= 7)", draft_k);
-    QB_REQUIRE(draft_k == 0 || m->cfg.mtp_layers == 1, "draft depth > 0 needs the MTP layer");
-    QB_CUDA(cudaSetDevice(ctx->device));
+// Caches, recurrent state and activations of the qwen35 family.
+static int qwen35_batch_alloc(qb_ctx *ctx, qb_batch *b, size_t slots) {
+    qb_model *m = b->m;
     const qb_model_config &c = m->cfg;
-    qb_batch *b = new qb_batch();
-    b->m = m; b->n_seqs = n_seqs; b->n_active = n_seqs; b->max_ctx = max_ctx; b->k = draft_k; b->page_size = page_size;
-    b->pages_per_seq = (max_ctx + draft_k + 1 + page_size - 1) / page_size;
-    b->chunk = std::max(1u, env_u32("QW3B200_PREFILL_CHUNK", 512));
+    const uint32_t n_seqs = b->n_seqs, max_ctx = b->max_ctx, draft_k = b->k, page_size = b->page_size;
+    const uint32_t H = c.n_embd, K1 = draft_k + 1, L = c.n_layers, rows = b->rows_cap;
+    b->gemm_impl = (int)qb_env_u32("QW3B200_GEMM_IMPL", 0);
     // The tensor-memory attention kernel wins once a call has enough keys to fill the GPU (one long context, or many
     // sequences) and costs a few microseconds per call below that; the two kernels differ in the last bits, so the choice
     // is a property of the batch (the keys it can hold), the same for every row the batch ever computes.
-    b->attn_tc = (uint64_t)n_seqs * max_ctx >= env_u32("QW3B200_ATTN_TC_MIN_KEYS", 16384);
+    b->attn_tc = (uint64_t)n_seqs * max_ctx >= qb_env_u32("QW3B200_ATTN_TC_MIN_KEYS", 16384);
     // Splits of 256 keys where the tensor-memory kernel runs (its tile pair); 128 keys otherwise: a short context then
     // spreads over twice the SMs, each streaming half the K/V bytes (7.87 against 8.01 ms per step at 2 K context).
     {
         const bool tc_shape = (c.head_dim == 256 || c.head_dim == 128) && page_size == 16 && c.n_heads / std::max(1u, c.n_kv_heads) <= 8;
-        b->attn_split = b->attn_tc && tc_shape ? 256 : env_u32("QW3B200_ATTN_SPLIT_SMALL", 128);
+        b->attn_split = b->attn_tc && tc_shape ? 256 : qb_env_u32("QW3B200_ATTN_SPLIT_SMALL", 128);
         if (b->attn_split < 64 || b->attn_split % 64) b->attn_split = 128;
     }
-    b->logit_rows = n_seqs * (draft_k + 1);
-    b->rows_cap = std::max(b->chunk, b->logit_rows);
-    b->gemm_impl = (int)env_u32("QW3B200_GEMM_IMPL", 0);
-    const uint32_t H = c.n_embd, K1 = draft_k + 1, L = c.n_layers, rows = b->rows_cap;
-    const size_t slots = (size_t)(pool_pages ? pool_pages : n_seqs * b->pages_per_seq) * page_size;
     const uint32_t kvd = m->kvd();
     b->kc.assign(L + 1, nullptr); b->vc.assign(L + 1, nullptr); b->state.assign(L, nullptr); b->conv.assign(L, nullptr); b->conv_alt.assign(L, nullptr);
     for (uint32_t il = 0; il <= L; ++il) {
@@ -502,8 +400,71 @@ static int batch_create(qb_ctx *ctx, qb_model *m, uint32_t n_seqs, uint32_t max_
             QB_CUDA(cudaMemsetAsync(b->conv[il], 0, csz * sizeof(float), ctx->stream));
             QB_CUDA(cudaMalloc(&b->conv_alt[il], csz * sizeof(float)));
             QB_CUDA(cudaMemsetAsync(b->conv_alt[il], 0, csz * sizeof(float), ctx->stream));
+            // a sequence at a chunk end has its state in slot 0 and its conv window in slot 0 of the valid buffer
+            StateBlock sb, cb;
+            sb.buf[0] = b->state[il]; sb.per_seq = ssz / n_seqs; sb.head = ssz / n_seqs / K1;
+            cb.buf[0] = b->conv[il]; cb.buf[1] = b->conv_alt[il]; cb.per_seq = csz / n_seqs; cb.head = csz / n_seqs / K1;
+            b->blocks.push_back(sb); b->blocks.push_back(cb);
         }
     }
+    const uint32_t inner = m->inner(), vdim = m->vdim(), F = c.n_ff, V = c.vocab_size;
+    const uint32_t act_cols = std::max({m->attn_in(), m->dn_in(), 2 * F});
+    QB_CUDA(cudaMalloc(&b->mtp_h, (size_t)rows * H * sizeof(float)));
+    QB_CUDA(cudaMalloc(&b->embd, (size_t)rows * H * sizeof(float)));
+    QB_CUDA(cudaMalloc(&b->act, (size_t)rows * act_cols * sizeof(float)));
+    {
+        size_t per_row = 0;   // floats of split partials any GEMM of the model can need per row
+        auto consider = [&](uint32_t N, uint32_t K, bool always) {
+            const uint32_t S = qb_ksplit(N, K);
+            if (S > 1 || always) per_row = std::max(per_row, (size_t)S * N);
+        };
+        consider(m->attn_in(), H, true); consider(m->dn_in(), H, true); consider(2 * F, H, false); consider(V, H, false);
+        consider(H, inner, true); consider(H, vdim, true); consider(H, F, true); consider(H, 2 * H, true);
+        b->parts_floats = std::max<size_t>(per_row, 1) * rows;
+        QB_CUDA(cudaMalloc(&b->parts, b->parts_floats * sizeof(float)));
+    }
+    {
+        size_t ml = 0;
+        const size_t acc = qb_attention_scratch_floats(rows, c.n_heads, c.head_dim, max_ctx + draft_k + 1, &ml, b->attn_split);
+        QB_CUDA(cudaMalloc(&b->att_acc, acc * sizeof(float)));
+        QB_CUDA(cudaMalloc(&b->att_ml, ml * sizeof(float)));
+    }
+    QB_TRY(alloc_qbuf(b->xq_h, rows, H));
+    QB_TRY(alloc_qbuf(b->xq_attn, rows, inner));
+    QB_TRY(alloc_qbuf(b->xq_dn, rows, vdim));
+    QB_TRY(alloc_qbuf(b->xq_ffn, rows, F));
+    QB_TRY(alloc_qbuf(b->xq_cat, rows, 2 * H));
+    return QB_OK;
+}
+
+static void qwen35_batch_free(qb_batch *b) {
+    for (auto p : b->kc) if (p) cudaFree(p);
+    for (auto p : b->vc) if (p) cudaFree(p);
+    for (auto p : b->state) if (p) cudaFree(p);
+    for (auto p : b->conv) if (p) cudaFree(p);
+    for (auto p : b->conv_alt) if (p) cudaFree(p);
+    void *ptrs[] = {b->mtp_h, b->embd, b->act, b->parts, b->att_acc, b->att_ml, b->xq_h.q, b->xq_h.d, b->xq_attn.q,
+                    b->xq_attn.d, b->xq_dn.q, b->xq_dn.d, b->xq_ffn.q, b->xq_ffn.d, b->xq_cat.q, b->xq_cat.d, b->normed, b->tp_y};
+    for (void *p : ptrs) if (p) cudaFree(p);
+}
+
+extern "C" void qb_batch_destroy(qb_ctx *ctx, qb_batch *b);
+
+static int batch_create(qb_ctx *ctx, qb_model *m, uint32_t n_seqs, uint32_t max_ctx, uint32_t draft_k,
+                        uint32_t page_size, int page_order, uint32_t pool_pages, qb_batch **out) {
+    QB_REQUIRE(ctx && m && out && n_seqs > 0 && max_ctx > 0 && page_size > 0, "qb_batch_create: bad arguments");
+    QB_REQUIRE(draft_k <= 7, "draft depth %u unsupported (<= 7)", draft_k);
+    QB_REQUIRE(draft_k == 0 || m->cfg.mtp_layers == 1, "draft depth > 0 needs the MTP layer");
+    QB_CUDA(cudaSetDevice(ctx->device));
+    const qb_model_config &c = m->cfg;
+    qb_batch *b = new qb_batch();
+    b->m = m; b->n_seqs = n_seqs; b->n_active = n_seqs; b->max_ctx = max_ctx; b->k = draft_k; b->page_size = page_size;
+    b->pages_per_seq = (max_ctx + draft_k + 1 + page_size - 1) / page_size;
+    b->chunk = std::max(1u, qb_env_u32("QW3B200_PREFILL_CHUNK", m->arch->chunk));
+    b->logit_rows = n_seqs * (draft_k + 1);
+    b->rows_cap = std::max(b->chunk, b->logit_rows);
+    const uint32_t H = c.n_embd, K1 = draft_k + 1, rows = b->rows_cap;
+    const size_t slots = (size_t)(pool_pages ? pool_pages : n_seqs * b->pages_per_seq) * page_size;
     // page table: identity / reverse / seeded shuffle over the whole pool
     {
         const size_t total = (size_t)n_seqs * b->pages_per_seq;
@@ -554,38 +515,13 @@ static int batch_create(qb_ctx *ctx, qb_model *m, uint32_t n_seqs, uint32_t max_
         QB_CUDA(cudaStreamSynchronize(ctx->stream));
     }
     // activations
-    const uint32_t inner = m->inner(), vdim = m->vdim(), F = c.n_ff, V = c.vocab_size;
-    const uint32_t act_cols = std::max({m->attn_in(), m->dn_in(), 2 * F});
+    const uint32_t V = c.vocab_size;
     QB_CUDA(cudaMalloc(&b->hid, (size_t)(rows + n_seqs) * H * sizeof(float)));
     QB_CUDA(cudaMemsetAsync(b->hid, 0, (size_t)(rows + n_seqs) * H * sizeof(float), ctx->stream));
-    QB_CUDA(cudaMalloc(&b->mtp_h, (size_t)rows * H * sizeof(float)));
-    QB_CUDA(cudaMalloc(&b->embd, (size_t)rows * H * sizeof(float)));
-    QB_CUDA(cudaMalloc(&b->act, (size_t)rows * act_cols * sizeof(float)));
     QB_CUDA(cudaMalloc(&b->logits, (size_t)b->logit_rows * V * sizeof(float)));
     QB_CUDA(cudaMalloc(&b->am_val, (size_t)b->logit_rows * QB_ARGMAX_BLOCKS * sizeof(float)));
     QB_CUDA(cudaMalloc(&b->am_idx, (size_t)b->logit_rows * QB_ARGMAX_BLOCKS * sizeof(int32_t)));
-    {
-        size_t per_row = 0;   // floats of split partials any GEMM of the model can need per row
-        auto consider = [&](uint32_t N, uint32_t K, bool always) {
-            const uint32_t S = qb_ksplit(N, K);
-            if (S > 1 || always) per_row = std::max(per_row, (size_t)S * N);
-        };
-        consider(m->attn_in(), H, true); consider(m->dn_in(), H, true); consider(2 * F, H, false); consider(V, H, false);
-        consider(H, inner, true); consider(H, vdim, true); consider(H, F, true); consider(H, 2 * H, true);
-        b->parts_floats = std::max<size_t>(per_row, 1) * rows;
-        QB_CUDA(cudaMalloc(&b->parts, b->parts_floats * sizeof(float)));
-    }
-    {
-        size_t ml = 0;
-        const size_t acc = qb_attention_scratch_floats(rows, c.n_heads, c.head_dim, max_ctx + draft_k + 1, &ml, b->attn_split);
-        QB_CUDA(cudaMalloc(&b->att_acc, acc * sizeof(float)));
-        QB_CUDA(cudaMalloc(&b->att_ml, ml * sizeof(float)));
-    }
-    QB_TRY(alloc_qbuf(b->xq_h, rows, H));
-    QB_TRY(alloc_qbuf(b->xq_attn, rows, inner));
-    QB_TRY(alloc_qbuf(b->xq_dn, rows, vdim));
-    QB_TRY(alloc_qbuf(b->xq_ffn, rows, F));
-    QB_TRY(alloc_qbuf(b->xq_cat, rows, 2 * H));
+    if (const int st = m->arch->batch_alloc(ctx, b, slots); st != QB_OK) { qb_batch_destroy(ctx, b); return st; }
     b->host_pos.assign(n_seqs, 0);
     b->chunk_end_pos.assign(n_seqs, -1);
     QB_CUDA(cudaStreamSynchronize(ctx->stream));
@@ -611,15 +547,8 @@ extern "C" void qb_batch_destroy(qb_ctx *ctx, qb_batch *b) {
     if (!b) return;
     cudaStreamSynchronize(ctx->stream);
     delete b->pool;
-    for (auto p : b->kc) if (p) cudaFree(p);
-    for (auto p : b->vc) if (p) cudaFree(p);
-    for (auto p : b->state) if (p) cudaFree(p);
-    for (auto p : b->conv) if (p) cudaFree(p);
-    for (auto p : b->conv_alt) if (p) cudaFree(p);
-    void *ptrs[] = {b->page_table, b->ctl, b->stats, b->hid, b->mtp_h, b->embd, b->act, b->parts,
-                    b->logits, b->am_val, b->am_idx, b->att_acc, b->att_ml, b->xq_h.q, b->xq_h.d, b->xq_attn.q,
-                    b->xq_attn.d, b->xq_dn.q, b->xq_dn.d, b->xq_ffn.q, b->xq_ffn.d, b->xq_cat.q, b->xq_cat.d, b->samp_u, b->seen, b->swap_tmp,
-                    b->normed, b->tp_y};
+    b->m->arch->batch_free(b);
+    void *ptrs[] = {b->page_table, b->ctl, b->stats, b->hid, b->logits, b->am_val, b->am_idx, b->samp_u, b->seen, b->swap_tmp, b->score_logits, b->score_map};
     for (void *p : ptrs) if (p) cudaFree(p);
     if (b->out_rec_host) cudaFreeHost(b->out_rec_host);
     if (b->limit_host) cudaFreeHost(b->limit_host);
@@ -876,14 +805,6 @@ static int plain_norm_quant(qb_ctx *ctx, qb_batch *b, const float *x, const int3
     return qb_launch_norm_quant(ctx, a);
 }
 
-struct RowSet {
-    uint32_t seq0 = 0, ns = 0, R = 0;      // sequences [seq0, seq0+ns), R rows each
-    const int32_t *seq_pos = nullptr;      // device [ns]: position of each sequence's first row
-    uint32_t max_pos = 0;                  // host upper bound of any row position
-    bool ingest = false;                   // rows of a prompt chunk (not of a decode / verify step)
-    uint32_t rows() const { return ns * R; }
-};
-
 // One attention block on h (xq_h already holds quant(rmsnorm(h))).  kv_only: K/V append only.
 static int attention_block(qb_ctx *ctx, qb_batch *b, const LayerW &L, uint32_t cache_idx, float *h, const RowSet &rs, bool kv_only,
                            const float *next_norm_w) {
@@ -958,13 +879,10 @@ static int deltanet_block(qb_ctx *ctx, qb_batch *b, const LayerW &L, uint32_t il
     return residual_norm_quant(ctx, b, h, rows, S, next_norm_w, b->xq_h, 0, true, nullptr, b->tp ? b->normed : nullptr);
 }
 
-// Target model on a row set.  tokens on the device ([rows]).  Leaves the pre-output-norm hidden rows
-// in b->hid[0 .. rows).  logits: 0 none, 1 every row, 2 last row of each sequence.
-static int target_forward(qb_ctx *ctx, qb_batch *b, const int32_t *tokens_dev, const RowSet &rs, bool checkpoints, int logits) {
+static int qwen35_forward(qb_ctx *ctx, qb_batch *b, const int32_t *tokens_dev, const RowSet &rs, bool checkpoints) {
     qb_model *m = b->m;
     const qb_model_config &c = m->cfg;
     const uint32_t rows = rs.rows();
-    QB_REQUIRE(rows <= b->rows_cap, "forward: %u rows exceed capacity %u", rows, b->rows_cap);
     float *h = b->hid;
     QB_TRY(qb_launch_get_rows(ctx, m->token_embd, tokens_dev, rows, h, c.n_embd));
     QB_TRY(plain_norm_quant(ctx, b, h, nullptr, rows, m->layers[0].attn_norm, b->xq_h));
@@ -988,22 +906,36 @@ static int target_forward(qb_ctx *ctx, qb_batch *b, const int32_t *tokens_dev, c
                                     cudaMemcpyDeviceToDevice, ctx->stream));
         }
     }
+    return QB_OK;
+}
+
+// xq_h holds the normalised rows just forwarded; mapped rows are normalised and quantised again as a compact batch.
+static int qwen35_head(qb_ctx *ctx, qb_batch *b, const int32_t *row_map, uint32_t rows, float *dst) {
+    if (row_map) QB_TRY(plain_norm_quant(ctx, b, b->hid, row_map, rows, b->m->output_norm, b->xq_h));
+    return gemm_to(ctx, b, b->m->output, b->xq_h, rows, dst);
+}
+
+extern const QbArch ARCH_QWEN35 = {"qwen35", 512, qwen35_batch_alloc, qwen35_batch_free, qwen35_forward, qwen35_head, qwen35_model_free};
+
+// The model's layers on a row set.  tokens on the device ([rows]).  Leaves the pre-output-norm hidden rows
+// in b->hid[0 .. rows).  logits: 0 none, 1 every row, 2 last row of each sequence.
+static int target_forward(qb_ctx *ctx, qb_batch *b, const int32_t *tokens_dev, const RowSet &rs, bool checkpoints, int logits) {
+    const qb_model_config &c = b->m->cfg;
+    const uint32_t rows = rs.rows();
+    QB_REQUIRE(rows <= b->rows_cap, "forward: %u rows exceed capacity %u", rows, b->rows_cap);
+    QB_TRY(b->m->arch->forward(ctx, b, tokens_dev, rs, checkpoints));
     b->last_logit_rows = 0;
-    if (logits == 1) {
-        QB_REQUIRE(rows <= b->logit_rows, "logits for %u rows exceed capacity %u", rows, b->logit_rows);
-        QB_TRY(gemm_to(ctx, b, m->output, b->xq_h, rows, b->logits));
-        QB_TRY(qb_launch_argmax_partial(ctx, b->logits, rows, c.vocab_size, c.vocab_size, b->am_val, b->am_idx, QB_ARGMAX_BLOCKS));
-        b->last_logit_rows = rows;
-    } else if (logits == 2) {
-        // last row of each sequence: quantise those rows again as a compact batch
+    if (logits == 0) return QB_OK;
+    const uint32_t n = logits == 1 ? rows : rs.ns;
+    QB_REQUIRE(n <= b->logit_rows, "logits for %u rows exceed capacity %u", n, b->logit_rows);
+    if (logits == 2) {
         std::vector<int32_t> map(rs.ns);
         for (uint32_t s = 0; s < rs.ns; ++s) map[s] = (int32_t)(s * rs.R + rs.R - 1);
         QB_CUDA(cudaMemcpyAsync(b->map_last, map.data(), rs.ns * sizeof(int32_t), cudaMemcpyHostToDevice, ctx->stream));
-        QB_TRY(plain_norm_quant(ctx, b, h, b->map_last, rs.ns, m->output_norm, b->xq_h));
-        QB_TRY(gemm_to(ctx, b, m->output, b->xq_h, rs.ns, b->logits));
-        QB_TRY(qb_launch_argmax_partial(ctx, b->logits, rs.ns, c.vocab_size, c.vocab_size, b->am_val, b->am_idx, QB_ARGMAX_BLOCKS));
-        b->last_logit_rows = rs.ns;
     }
+    QB_TRY(b->m->arch->head(ctx, b, logits == 2 ? b->map_last : nullptr, n, b->logits));
+    QB_TRY(qb_launch_argmax_partial(ctx, b->logits, n, c.vocab_size, c.vocab_size, b->am_val, b->am_idx, QB_ARGMAX_BLOCKS));
+    b->last_logit_rows = n;
     return QB_OK;
 }
 
@@ -1169,11 +1101,12 @@ extern "C" int qb_seq_pages(qb_ctx *ctx, qb_batch *b, uint32_t seq, int32_t *pag
 // first token with it), the prefix's tokens (seen-token record).  Attaching it to an empty sequence makes that sequence
 // continue from the prefix end without ingesting it: same pages, copied state.  The prefix length must be a whole number
 // of pages, so the sequences' own tokens go to pages of their own.
+static float *valid_state(const qb_batch *b, const StateBlock &sb) { return sb.buf[1] && b->conv_par ? sb.buf[1] : sb.buf[0]; }
 struct qb_prefix {
     qb_batch *owner = nullptr;
     uint32_t n_tokens = 0;
     std::vector<int32_t> pages;
-    std::vector<float *> state, conv;     // per layer (recurrent layers only)
+    std::vector<float *> state;           // one copy per StateBlock of the batch
     float *hid = nullptr;
     int32_t *tokens_dev = nullptr;
 };
@@ -1187,7 +1120,6 @@ extern "C" void qb_prefix_release(qb_ctx *ctx, qb_prefix *px) {
     cudaStreamSynchronize(ctx->stream);
     for (auto it = px->pages.rbegin(); it != px->pages.rend(); ++it) px->owner->pool->drop(*it);
     for (float *p : px->state) if (p) cudaFree(p);
-    for (float *p : px->conv) if (p) cudaFree(p);
     if (px->hid) cudaFree(px->hid);
     if (px->tokens_dev) cudaFree(px->tokens_dev);
     delete px;
@@ -1203,20 +1135,14 @@ extern "C" int qb_prefix_capture(qb_ctx *ctx, qb_batch *b, uint32_t seq, const i
     QB_REQUIRE(tokens_host || !b->seen, "qb_prefix_capture: a batch with token penalties needs the prefix's tokens");
     QB_CUDA(cudaSetDevice(ctx->device));
     const qb_model_config &c = b->m->cfg;
-    const uint32_t K1 = b->k + 1;
-    const size_t sfl = (size_t)c.ssm_num_v_heads * c.ssm_head_dim * c.ssm_head_dim, cfl = (size_t)b->m->qkv_dim() * 3;
     qb_prefix *px = new qb_prefix();
     px->owner = b; px->n_tokens = (uint32_t)n;
-    px->state.assign(c.n_layers, nullptr); px->conv.assign(c.n_layers, nullptr);
+    px->state.assign(b->blocks.size(), nullptr);
     auto fail = [&](int st) { qb_prefix_release(ctx, px); return st; };
-    for (uint32_t il = 0; il < c.n_layers; ++il) {
-        if (!b->state[il]) continue;
-        // a sequence at a chunk end has its state in slot 0 and its conv window in slot 0 of the valid buffer
-        if (cudaMalloc(&px->state[il], sfl * sizeof(float)) != cudaSuccess || cudaMalloc(&px->conv[il], cfl * sizeof(float)) != cudaSuccess)
-            return fail(qb_fail(QB_ERR_CUDA, "qb_prefix_capture: out of device memory"));
-        const float *cv = b->conv_par ? b->conv_alt[il] : b->conv[il];
-        QB_CUDA(cudaMemcpyAsync(px->state[il], b->state[il] + (size_t)seq * K1 * sfl, sfl * sizeof(float), cudaMemcpyDeviceToDevice, ctx->stream));
-        QB_CUDA(cudaMemcpyAsync(px->conv[il], cv + (size_t)seq * K1 * cfl, cfl * sizeof(float), cudaMemcpyDeviceToDevice, ctx->stream));
+    for (size_t i = 0; i < b->blocks.size(); ++i) {
+        const StateBlock &sb = b->blocks[i];
+        if (cudaMalloc(&px->state[i], sb.head * sizeof(float)) != cudaSuccess) return fail(qb_fail(QB_ERR_CUDA, "qb_prefix_capture: out of device memory"));
+        QB_CUDA(cudaMemcpyAsync(px->state[i], valid_state(b, sb) + (size_t)seq * sb.per_seq, sb.head * sizeof(float), cudaMemcpyDeviceToDevice, ctx->stream));
     }
     QB_CUDA(cudaMalloc(&px->hid, (size_t)c.n_embd * sizeof(float)));
     QB_CUDA(cudaMemcpyAsync(px->hid, b->hid + (size_t)(b->rows_cap + seq) * c.n_embd, (size_t)c.n_embd * sizeof(float), cudaMemcpyDeviceToDevice, ctx->stream));
@@ -1243,17 +1169,14 @@ extern "C" int qb_prefix_attach(qb_ctx *ctx, qb_batch *b, uint32_t seq, const qb
     QB_CUDA(cudaSetDevice(ctx->device));
     const qb_model_config &c = b->m->cfg;
     const uint32_t K1 = b->k + 1;
-    const size_t sfl = (size_t)c.ssm_num_v_heads * c.ssm_head_dim * c.ssm_head_dim, cfl = (size_t)b->m->qkv_dim() * 3;
     for (int32_t pg : px->pages) {
         QB_REQUIRE(b->pool->share(pg), "qb_prefix_attach: page %d of the prefix is not in use", pg);
         b->seq_pages[seq].push_back(pg);
     }
     QB_TRY(upload_pages(ctx, b, seq, 0, (uint32_t)px->pages.size()));
-    for (uint32_t il = 0; il < c.n_layers; ++il) {
-        if (!b->state[il]) continue;
-        float *cv = b->conv_par ? b->conv_alt[il] : b->conv[il];
-        QB_CUDA(cudaMemcpyAsync(b->state[il] + (size_t)seq * K1 * sfl, px->state[il], sfl * sizeof(float), cudaMemcpyDeviceToDevice, ctx->stream));
-        QB_CUDA(cudaMemcpyAsync(cv + (size_t)seq * K1 * cfl, px->conv[il], cfl * sizeof(float), cudaMemcpyDeviceToDevice, ctx->stream));
+    for (size_t i = 0; i < b->blocks.size(); ++i) {
+        const StateBlock &sb = b->blocks[i];
+        QB_CUDA(cudaMemcpyAsync(valid_state(b, sb) + (size_t)seq * sb.per_seq, px->state[i], sb.head * sizeof(float), cudaMemcpyDeviceToDevice, ctx->stream));
     }
     QB_CUDA(cudaMemcpyAsync(b->hid + (size_t)(b->rows_cap + seq) * c.n_embd, px->hid, (size_t)c.n_embd * sizeof(float), cudaMemcpyDeviceToDevice, ctx->stream));
     QB_CUDA(qb_launch_pdl(ctx->stream, set_seq_ctl_kernel, dim3(1), dim3(32), (size_t)0, b->pos, b->sel, b->cur,
@@ -1271,8 +1194,41 @@ extern "C" int qb_prefix_attach(qb_ctx *ctx, qb_batch *b, uint32_t seq, const qb
 }
 extern "C" uint32_t qb_prefix_tokens(const qb_prefix *px) { return px ? px->n_tokens : 0; }
 
+// Logits of chosen rows of a prompt part (qb_prefill_logits).
+struct WantedRows { const int32_t *at; uint32_t n; float *host; };
+static constexpr uint32_t SCORE_ROWS = 64;
+// ... of the chunk [off, off + M) just forwarded, in groups of SCORE_ROWS rows.
+static int wanted_logits(qb_ctx *ctx, qb_batch *b, const WantedRows &w, uint32_t off, uint32_t M) {
+    const uint32_t V = b->m->cfg.vocab_size, cap = std::min(SCORE_ROWS, b->rows_cap);
+    if (!b->score_logits) {
+        QB_CUDA(cudaMalloc(&b->score_logits, (size_t)cap * V * sizeof(float)));
+        QB_CUDA(cudaMalloc(&b->score_map, (size_t)cap * sizeof(int32_t)));
+    }
+    std::vector<int32_t> map;
+    std::vector<uint32_t> dst;
+    auto flush = [&]() -> int {
+        if (map.empty()) return QB_OK;
+        QB_CUDA(cudaMemcpyAsync(b->score_map, map.data(), map.size() * sizeof(int32_t), cudaMemcpyHostToDevice, ctx->stream));
+        QB_TRY(b->m->arch->head(ctx, b, b->score_map, (uint32_t)map.size(), b->score_logits));
+        for (size_t i = 0; i < dst.size(); ++i)
+            QB_CUDA(cudaMemcpyAsync(w.host + (size_t)dst[i] * V, b->score_logits + i * V, (size_t)V * sizeof(float), cudaMemcpyDeviceToHost, ctx->stream));
+        QB_CUDA(cudaStreamSynchronize(ctx->stream));
+        map.clear();
+        dst.clear();
+        return QB_OK;
+    };
+    for (uint32_t i = 0; i < w.n; ++i) {
+        const uint32_t at = (uint32_t)w.at[i];
+        if (at < off || at >= off + M) continue;
+        map.push_back((int32_t)(at - off));
+        dst.push_back(i);
+        if (map.size() == cap) QB_TRY(flush());
+    }
+    return flush();
+}
+
 static int prefill_impl(qb_ctx *ctx, qb_batch *b, uint32_t seq, const int32_t *tokens_host, uint32_t n, bool more_follows,
-                        const qb_sampling *samp) {
+                        const qb_sampling *samp, const WantedRows *want = nullptr) {
     QB_REQUIRE(ctx && b && tokens_host && n > 0 && seq < b->n_seqs, "qb_prefill: bad arguments");
     QB_REQUIRE((uint32_t)b->host_pos[seq] + n <= b->max_ctx, "qb_prefill: %u tokens at position %d exceed max_ctx %u", n, b->host_pos[seq],
                b->max_ctx);
@@ -1318,6 +1274,7 @@ static int prefill_impl(qb_ctx *ctx, qb_batch *b, uint32_t seq, const int32_t *t
         RowSet rs;
         rs.seq0 = seq; rs.ns = 1; rs.R = M; rs.seq_pos = b->pos + seq; rs.max_pos = p0 + M; rs.ingest = true;
         QB_TRY(target_forward(ctx, b, toks, rs, false, last ? 2 : 0));
+        if (want) QB_TRY(wanted_logits(ctx, b, *want, off, M));
         if (c.mtp_layers && b->k > 0) {
             // MTP-layer K/V of the chunk: row r pairs token r with the target hidden of row r-1 (row 0: the previous chunk's
             // last hidden, kept behind the chunk rows)
@@ -1362,6 +1319,16 @@ extern "C" int qb_prefill_chunk(qb_ctx *ctx, qb_batch *b, uint32_t seq, const in
     return prefill_impl(ctx, b, seq, tokens_host, n, true, nullptr);
 }
 
+// The same, scoring chosen positions: logits_host[i] = the logits at token want[i] of this part.
+extern "C" int qb_prefill_logits(qb_ctx *ctx, qb_batch *b, uint32_t seq, const int32_t *tokens_host, uint32_t n, const int32_t *want, uint32_t n_want,
+                                 float *logits_host) {
+    QB_REQUIRE(n_want == 0 || (want && logits_host), "qb_prefill_logits: null argument");
+    for (uint32_t i = 0; i < n_want; ++i) QB_REQUIRE(want[i] >= 0 && (uint32_t)want[i] < n, "qb_prefill_logits: place %d of %u tokens", want[i], n);
+    const WantedRows w{want, n_want, logits_host};
+    QB_TRY(prefill_impl(ctx, b, seq, tokens_host, n, true, nullptr, n_want ? &w : nullptr));
+    return n_want ? qb_synchronize(ctx) : QB_OK;
+}
+
 // The end of a sampled request's prompt: the first token is drawn with the request's first uniform draw u.
 extern "C" int qb_prefill_sampled(qb_ctx *ctx, qb_batch *b, uint32_t seq, const int32_t *tokens_host, uint32_t n, const qb_sampling *samp,
                                   double u) {
@@ -1381,8 +1348,28 @@ static int check_room(qb_batch *b, uint32_t need) {
     return QB_OK;
 }
 
-extern "C" int qb_decode_greedy_step(qb_ctx *ctx, qb_batch *b) {
-    QB_REQUIRE(ctx && b, "qb_decode_greedy_step: null argument");
+// The step's draws go through a pinned ring, no stream synchronisation: a slot waits only for its own copy of four steps ago.
+static int stage_draws(qb_ctx *ctx, qb_batch *b, double **u) {
+    const size_t n = 2 * (size_t)b->n_seqs * (b->k + 1);
+    if (!b->samp_u) QB_CUDA(cudaMalloc(&b->samp_u, n * sizeof(double)));
+    if (!b->samp_stage) {
+        QB_CUDA(cudaHostAlloc(&b->samp_stage, qb_batch::SAMP_RING * n * sizeof(double), cudaHostAllocDefault));
+        for (cudaEvent_t &e : b->samp_ev) QB_CUDA(cudaEventCreateWithFlags(&e, cudaEventDisableTiming));
+    }
+    b->samp_slot = (b->samp_slot + 1) % qb_batch::SAMP_RING;
+    QB_CUDA(cudaEventSynchronize(b->samp_ev[b->samp_slot]));
+    *u = b->samp_stage + b->samp_slot * n;
+    return QB_OK;
+}
+static int send_draws(qb_ctx *ctx, qb_batch *b, const double *u, size_t n) {
+    QB_CUDA(cudaMemcpyAsync(b->samp_u, u, n * sizeof(double), cudaMemcpyHostToDevice, ctx->stream));
+    QB_CUDA(cudaEventRecord(b->samp_ev[b->samp_slot], ctx->stream));
+    return QB_OK;
+}
+
+// One plain step of every active sequence; the row's token is its argmax, or what `pick` leaves in its place.
+template <typename Pick>
+static int decode_step(qb_ctx *ctx, qb_batch *b, Pick pick) {
     QB_TRY(check_room(b, 1));
     QB_CUDA(cudaSetDevice(ctx->device));
     QB_TRY(ensure_step_pages(ctx, b, 1));
@@ -1390,6 +1377,7 @@ extern "C" int qb_decode_greedy_step(qb_ctx *ctx, qb_batch *b) {
     RowSet rs;
     rs.seq0 = 0; rs.ns = b->n_active; rs.R = 1; rs.seq_pos = b->pos; rs.max_pos = max_host_pos(b) + 1;
     QB_TRY(target_forward(ctx, b, b->cur, rs, false, 1));
+    QB_TRY(pick());
     QB_CUDA(qb_launch_pdl(ctx->stream, greedy_commit_kernel, dim3(b->n_active), dim3(256), (size_t)(0), b->am_val, b->am_idx, 0, 0, 1, 0, b->n_active, b->k + 1, b->rows_cap,
                                                            c.n_embd, b->pos, b->sel, b->cur, 1, b->out_rec, b->n_seqs, b->hid,
                                                            (unsigned long long *)b->stats));
@@ -1397,6 +1385,31 @@ extern "C" int qb_decode_greedy_step(qb_ctx *ctx, qb_batch *b) {
     QB_TRY(mark_seen_record(ctx, b, 0, b->n_active));
     advance_host_pos(b, 1);
     return probe_tick(ctx, b);
+}
+
+extern "C" int qb_decode_greedy_step(qb_ctx *ctx, qb_batch *b) {
+    QB_REQUIRE(ctx && b, "qb_decode_greedy_step: null argument");
+    return decode_step(ctx, b, []() { return QB_OK; });
+}
+
+// A plain sampled step: sequence s draws its token from the row's truncated distribution with u_host[s].
+extern "C" int qb_decode_sampled_step(qb_ctx *ctx, qb_batch *b, const qb_sampling *samp, const double *u_host) {
+    QB_REQUIRE(ctx && b && samp && u_host && samp->temp > 0.0f, "qb_decode_sampled_step: needs draws and temp > 0");
+    const uint32_t V = b->m->cfg.vocab_size;
+    return decode_step(ctx, b, [&]() -> int {
+        double *u = nullptr;
+        QB_TRY(stage_draws(ctx, b, &u));
+        for (uint32_t s = 0; s < b->n_active; ++s) u[s] = u_host[s];
+        QB_TRY(send_draws(ctx, b, u, b->n_active));
+        for (uint32_t s = 0; s < (b->seen ? b->n_active : 1u); ++s) {       // token penalties: a record per sequence
+            const uint32_t rows = b->seen ? 1 : b->n_active;
+            QB_TRY(qb_launch_sample_rows(ctx, b->logits + (size_t)s * V, rows, V, V, nullptr, 0, b->samp_u + s, b->samp_u + s, samp->temp, samp->top_p,
+                                         samp->top_k, samp->min_p, nullptr, nullptr, nullptr, b->am_val + (size_t)s * QB_ARGMAX_BLOCKS,
+                                         b->am_idx + (size_t)s * QB_ARGMAX_BLOCKS, QB_ARGMAX_BLOCKS, b->pen_presence, b->pen_repetition,
+                                         b->seen ? b->seen + (size_t)s * b->seen_words : nullptr, b->seen_words));
+        }
+        return QB_OK;
+    });
 }
 
 extern "C" int qb_mtp_draft(qb_ctx *ctx, qb_batch *b) {
@@ -1471,7 +1484,7 @@ extern "C" int qb_mtp_accept_commit(qb_ctx *ctx, qb_batch *b) {
 // same calls on the same tokens; all of them get the same bits.  NULL goes back to the single-GPU form.
 extern "C" int qb_batch_set_tp(qb_ctx *ctx, qb_batch *b, qb_tp_group *group) {
     QB_REQUIRE(ctx && b, "qb_batch_set_tp: null argument");
-    QB_REQUIRE(!group || b->m->tp_world > 1 || b->m->tp_world == 1, "qb_batch_set_tp: bad model");
+    QB_REQUIRE(!group || !b->layered, "qb_batch_set_tp: the %s family has no sharded form", b->m->arch->name);
     if (group && !b->normed) {
         const size_t n = (size_t)b->rows_cap * b->m->cfg.n_embd * sizeof(float);
         QB_CUDA(cudaMalloc(&b->normed, n));
@@ -1508,23 +1521,14 @@ extern "C" int qb_mtp_sample_rows(qb_ctx *ctx, qb_batch *b, float temp, float to
     QB_REQUIRE(ctx && b && u_host && b->k > 0, "qb_mtp_sample_rows: needs draws and a batch with draft depth > 0");
     QB_CUDA(cudaSetDevice(ctx->device));
     const uint32_t ns = b->n_active, k = b->k, K1 = k + 1, rows = ns * K1;
-    if (!b->samp_u) QB_CUDA(cudaMalloc(&b->samp_u, 2 * (size_t)b->n_seqs * K1 * sizeof(double)));
-    const size_t slot_doubles = 2 * (size_t)b->n_seqs * K1;
-    if (!b->samp_stage) {
-        QB_CUDA(cudaHostAlloc(&b->samp_stage, qb_batch::SAMP_RING * slot_doubles * sizeof(double), cudaHostAllocDefault));
-        for (cudaEvent_t &e : b->samp_ev) QB_CUDA(cudaEventCreateWithFlags(&e, cudaEventDisableTiming));
-    }
-    // no stream synchronisation: the draws go through a pinned ring; a slot waits only for its own copy of four steps ago
-    const uint32_t slot = b->samp_slot++ % qb_batch::SAMP_RING;
-    QB_CUDA(cudaEventSynchronize(b->samp_ev[slot]));
-    double *u = b->samp_stage + slot * slot_doubles;
+    double *u = nullptr;
+    QB_TRY(stage_draws(ctx, b, &u));
     for (uint32_t s = 0; s < ns; ++s)
         for (uint32_t i = 0; i < K1; ++i) {
             u[(size_t)s * K1 + i] = u_host[(size_t)s * K1 + i];                                  // acceptance draw of row i
             u[(size_t)rows + s * K1 + i] = u_host[(size_t)s * K1 + (i < k ? i + 1 : k)];          // residual / bonus draw
         }
-    QB_CUDA(cudaMemcpyAsync(b->samp_u, u, 2 * (size_t)rows * sizeof(double), cudaMemcpyHostToDevice, ctx->stream));
-    QB_CUDA(cudaEventRecord(b->samp_ev[slot], ctx->stream));
+    QB_TRY(send_draws(ctx, b, u, 2 * (size_t)rows));
     const qb_model_config &c = b->m->cfg;
     return qb_launch_sample_rows(ctx, b->logits, rows, c.vocab_size, c.vocab_size, b->drafts, K1, b->samp_u, b->samp_u + rows, temp, top_p,
                                  top_k, min_p, nullptr, nullptr, nullptr, b->am_val, b->am_idx, QB_ARGMAX_BLOCKS, b->pen_presence, b->pen_repetition,
@@ -1591,13 +1595,9 @@ extern "C" int qb_seq_reset(qb_ctx *ctx, qb_batch *b, uint32_t seq) {
     QB_CUDA(cudaSetDevice(ctx->device));
     const qb_model_config &c = b->m->cfg;
     const uint32_t K1 = b->k + 1;
-    const size_t ssz = (size_t)K1 * c.ssm_num_v_heads * c.ssm_head_dim * c.ssm_head_dim, csz = (size_t)K1 * b->m->qkv_dim() * 3;
-    for (uint32_t il = 0; il < c.n_layers; ++il) {
-        if (!b->state[il]) continue;
-        QB_CUDA(cudaMemsetAsync(b->state[il] + seq * ssz, 0, ssz * sizeof(float), ctx->stream));
-        QB_CUDA(cudaMemsetAsync(b->conv[il] + seq * csz, 0, csz * sizeof(float), ctx->stream));
-        QB_CUDA(cudaMemsetAsync(b->conv_alt[il] + seq * csz, 0, csz * sizeof(float), ctx->stream));
-    }
+    for (const StateBlock &sb : b->blocks)
+        for (float *p : sb.buf)
+            if (p) QB_CUDA(cudaMemsetAsync(p + seq * sb.per_seq, 0, sb.per_seq * sizeof(float), ctx->stream));
     // the step record of the slot too: the host's position mirror is refreshed from it (qb_read_step_output)
     for (int32_t *p : {b->pos, b->sel, b->cur, b->prefix_pos, b->out_rec, b->out_rec + b->n_seqs + (size_t)b->n_seqs * K1})
         QB_CUDA(cudaMemsetAsync(p + seq, 0, sizeof(int32_t), ctx->stream));
@@ -1627,10 +1627,8 @@ extern "C" int qb_seq_swap(qb_ctx *ctx, qb_batch *b, uint32_t s1, uint32_t s2) {
     QB_CUDA(cudaSetDevice(ctx->device));
     const qb_model_config &c = b->m->cfg;
     const uint32_t K1 = b->k + 1;
-    const size_t ssz = (size_t)K1 * c.ssm_num_v_heads * c.ssm_head_dim * c.ssm_head_dim * sizeof(float);
-    const size_t csz = (size_t)K1 * b->m->qkv_dim() * 3 * sizeof(float);
-    const size_t need = std::max({ssz, csz, (size_t)c.n_embd * sizeof(float), (size_t)b->pages_per_seq * sizeof(int32_t),
-                                  (size_t)b->seen_words * sizeof(uint32_t)});
+    size_t need = std::max({(size_t)c.n_embd * sizeof(float), (size_t)b->pages_per_seq * sizeof(int32_t), (size_t)b->seen_words * sizeof(uint32_t)});
+    for (const StateBlock &sb : b->blocks) need = std::max(need, sb.per_seq * sizeof(float));
     if (b->swap_bytes < need) {
         if (b->swap_tmp) { QB_CUDA(cudaStreamSynchronize(ctx->stream)); QB_CUDA(cudaFree(b->swap_tmp)); b->swap_tmp = nullptr; }
         QB_CUDA(cudaMalloc(&b->swap_tmp, need));
@@ -1643,12 +1641,9 @@ extern "C" int qb_seq_swap(qb_ctx *ctx, qb_batch *b, uint32_t s1, uint32_t s2) {
         QB_CUDA(cudaMemcpyAsync(d, b->swap_tmp, bytes, cudaMemcpyDeviceToDevice, ctx->stream));
         return QB_OK;
     };
-    for (uint32_t il = 0; il < c.n_layers; ++il) {
-        if (!b->state[il]) continue;
-        QB_TRY(swap_block(b->state[il], ssz));
-        QB_TRY(swap_block(b->conv[il], csz));
-        QB_TRY(swap_block(b->conv_alt[il], csz));
-    }
+    for (const StateBlock &sb : b->blocks)
+        for (float *p : sb.buf)
+            if (p) QB_TRY(swap_block(p, sb.per_seq * sizeof(float)));
     QB_TRY(swap_block(b->page_table, (size_t)b->pages_per_seq * sizeof(int32_t)));
     QB_TRY(swap_block(b->hid + (size_t)b->rows_cap * c.n_embd, (size_t)c.n_embd * sizeof(float)));
     if (b->seen) QB_TRY(swap_block(b->seen, (size_t)b->seen_words * sizeof(uint32_t)));
@@ -1683,19 +1678,13 @@ static size_t ctl_count(const qb_batch *b) {
 template <typename F>
 static int for_each_state_block(qb_batch *b, F f) {
     const qb_model_config &c = b->m->cfg;
-    const uint32_t K1 = b->k + 1;
-    const size_t ssz = (size_t)b->n_seqs * K1 * c.ssm_num_v_heads * c.ssm_head_dim * c.ssm_head_dim * sizeof(float);
-    const size_t csz = (size_t)b->n_seqs * K1 * b->m->qkv_dim() * 3 * sizeof(float);
     QB_TRY(f((void *)b->ctl, ctl_count(b) * sizeof(int32_t)));
     QB_TRY(f((void *)(b->hid + (size_t)b->rows_cap * c.n_embd), (size_t)b->n_seqs * c.n_embd * sizeof(float)));
     QB_TRY(f((void *)b->stats, QB_STATS * sizeof(long long)));
     QB_TRY(f((void *)b->page_table, (size_t)b->n_seqs * b->pages_per_seq * sizeof(int32_t)));      // qb_seq_swap exchanges rows
-    for (uint32_t il = 0; il < c.n_layers; ++il) {
-        if (!b->state[il]) continue;
-        QB_TRY(f((void *)b->state[il], ssz));
-        QB_TRY(f((void *)b->conv[il], csz));
-        QB_TRY(f((void *)b->conv_alt[il], csz));
-    }
+    for (const StateBlock &sb : b->blocks)
+        for (float *p : sb.buf)
+            if (p) QB_TRY(f((void *)p, (size_t)b->n_seqs * sb.per_seq * sizeof(float)));
     if (b->seen) QB_TRY(f((void *)b->seen, (size_t)b->n_seqs * b->seen_words * sizeof(uint32_t)));
     return QB_OK;
 }
@@ -1752,4 +1741,34 @@ extern "C" int qb_debug_last_drafts(qb_ctx *ctx, qb_batch *b, int32_t *host_out)
     QB_CUDA(cudaMemcpyAsync(host_out, b->drafts, (size_t)b->n_seqs * b->k * sizeof(int32_t), cudaMemcpyDeviceToHost, ctx->stream));
     QB_CUDA(cudaStreamSynchronize(ctx->stream));
     return QB_OK;
+}
+
+// ---- model folders: config.json names the architecture -----------------------------------------------------------------
+static const QbLoader LOADERS[] = {
+    {"Kezilix", qb_layered_load},
+};
+
+extern "C" int qb_model_load(qb_ctx *ctx, const char *path, int f32, qb_model **out, qb_model_config *cfg_out) {
+    QB_REQUIRE(ctx && path && out, "qb_model_load: null argument");
+    struct stat st;
+    if (stat(path, &st) != 0) return qb_fail(QB_ERR_INVALID, "model: %s does not exist", path);
+    if (!S_ISDIR(st.st_mode)) {
+        if (f32) return qb_fail(QB_ERR_UNSUPPORTED, "model: the %s family computes on quantised weights and has no 32-bit form", ARCH_QWEN35.name);
+        return qb_model_load_gguf(ctx, path, out, cfg_out);
+    }
+    std::ifstream in(std::string(path) + "/config.json");
+    std::stringstream text;
+    if (!in || !(text << in.rdbuf())) return qb_fail(QB_ERR_INVALID, "model: cannot read %s/config.json", path);
+    const std::string config = text.str();
+    qbjson::Value root;
+    if (!qbjson::Parser(config.data(), config.size()).parse(root)) return qb_fail(QB_ERR_INVALID, "model: %s/config.json is not JSON", path);
+    const qbjson::Value *a = root.get("architecture");
+    const std::string name = a ? a->s : std::string();
+    for (const QbLoader &l : LOADERS)
+        if (name == l.architecture) {
+            QB_TRY(l.load(ctx, path, config, f32 != 0, out));
+            if (cfg_out) *cfg_out = (*out)->cfg;
+            return QB_OK;
+        }
+    return qb_fail(QB_ERR_UNSUPPORTED, "model: architecture '%s' is not known", name.c_str());
 }

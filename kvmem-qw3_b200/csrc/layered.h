@@ -1,0 +1,120 @@
+// Layered models: decoders described layer by layer in a config.json (mixer type and sizes, feed-forward, an optional loop
+// over a span of layers), with dense bfloat16 weights.  Mechanisms (retention.cu, latent_attention.cu, dense_gemm.cu,
+// layered_norm.cu) take their constants as arguments; layered_model.cu composes them.
+#pragma once
+
+#include "dense_gemm.h"
+
+// A rotary embedding on the device: pair i of the first `dims` dimensions turns by position * freq[i]; cos and sin are
+// multiplied by amp.  interleaved: pairs (2i, 2i + 1), else (i, i + dims / 2).
+struct QbRotary {
+    const float *freq = nullptr;
+    float amp = 1.0f;
+    uint32_t dims = 0;
+    bool interleaved = false;
+};
+
+#ifdef __CUDACC__
+template <typename T> __device__ __forceinline__ T qb_cast(float v);
+template <> __device__ __forceinline__ float qb_cast<float>(float v) { return v; }
+template <> __device__ __forceinline__ __nv_bfloat16 qb_cast<__nv_bfloat16>(float v) { return __float2bfloat16(v); }
+__device__ __forceinline__ float qb_f32(float v) { return v; }
+__device__ __forceinline__ float qb_f32(__nv_bfloat16 v) { return __bfloat162float(v); }
+// 32-bit angles: cos and sin of pair i at a position
+__device__ __forceinline__ void qb_rot_angle(const QbRotary &r, int pos, uint32_t i, float &c, float &s) {
+    sincosf((float)pos * r.freq[i], &s, &c);
+    c *= r.amp;
+    s *= r.amp;
+}
+// element j of a rotated vector: its pair index, its partner, and whether it is the first of the pair
+__device__ __forceinline__ void qb_rot_pair(const QbRotary &r, uint32_t j, uint32_t &i, uint32_t &partner, bool &first) {
+    if (r.interleaved) { i = j >> 1; partner = j ^ 1; first = !(j & 1); }
+    else { const uint32_t h = r.dims / 2; first = j < h; i = first ? j : j - h; partner = first ? j + h : j - h; }
+}
+// Sum over a block of `nwarps` warps; every thread returns it.  red: nwarps floats of shared memory.
+__device__ __forceinline__ float qb_block_sum(float v, float *red, uint32_t nwarps) {
+    v = warp_sum(v);
+    __syncthreads();
+    if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
+    __syncthreads();
+    float t = 0.0f;
+    for (uint32_t i = 0; i < nwarps; ++i) t += red[i];
+    return t;
+}
+#endif
+
+// ---- residual, loop additions and norm in one launch (layered_norm.cu) ------------------------------------------------
+struct QbLayerNorm {
+    uint32_t M = 0, n = 0;
+    float eps = 0.0f;
+    float *x = nullptr;                       // residual stream [M][n]
+    // source of the row: an embedding row (normalised with embed_w), or x + sum of parts
+    const int32_t *tokens = nullptr;
+    const __nv_bfloat16 *embed = nullptr;     // [vocab][n]
+    const float *embed_w = nullptr;
+    uint32_t vocab = 0;
+    const float *parts = nullptr;             // [S][M][n]
+    uint32_t S = 0;
+    const int32_t *row_map = nullptr;         // source rows of x (the stream is not written then)
+    float *trace = nullptr;                   // copy of the residual before the loop's additions [M][n]
+    float *emb_store = nullptr;               // the embedding output is kept here [M][n]
+    const float *emb_add = nullptr;           // ... and added
+    const float *step = nullptr;              // vector [n] added to every row
+    const float *w = nullptr;                 // gain of the norm that follows; null: no output
+    QbActBuf out;
+};
+int qb_launch_layer_norm(qb_ctx *ctx, const QbLayerNorm &a);
+
+// ---- retention (retention.cu) -------------------------------------------------------------------------------------------
+// Linear attention with one fixed decay per head: S_t = decay S_(t-1) + k_t v_t^T, o_t = S_t^T q_t, o divided by its root
+// mean square and gated by silu(g).  Rows are grouped per sequence (R rows each, consecutive positions).
+static const uint32_t QB_RET_CHUNK = 64;
+struct QbRetention {
+    float *proj = nullptr;                    // [S][rows][stride]: q (H*dim) | k (H*dim) | v (H*vdim) | g (H*vdim)
+    uint32_t S = 1, stride = 0;
+    uint32_t ns = 0, R = 0, H = 0, dim = 0, vdim = 0;
+    float eps = 0.0f;
+    QbRotary rot;
+    const float *powers = nullptr;            // [H][QB_RET_CHUNK + 1]: decay^0 .. decay^64
+    const int32_t *seq_pos = nullptr;
+    float *state = nullptr;                   // [ns][H][dim][vdim]
+    QbActBuf out;                             // [rows][H*vdim]
+};
+int qb_launch_retention(qb_ctx *ctx, const QbRetention &a);
+
+// ---- latent attention (latent_attention.cu) ----------------------------------------------------------------------------
+// Keys and values of all heads come from one latent vector per token; the cache holds the latent and one rotated key part
+// shared by the heads.  Few rows: the key projection is absorbed into the query and attention runs over the latents
+// themselves.  Prompt chunks: keys and values are expanded head by head first.
+struct QbLatent {
+    const float *proj = nullptr;              // [S][rows][stride]: q (H*(dim+rot_dim)) | latent (rank) | shared key part (rot_dim)
+    uint32_t S = 1, stride = 0;
+    uint32_t ns = 0, R = 0, H = 0, dim = 0, rot_dim = 0, vdim = 0, rank = 0;
+    float eps = 0.0f, scale = 1.0f;
+    QbRotary rot;
+    const float *norm_w = nullptr, *sink = nullptr;      // [rank], [H]
+    const QbDense *ukv = nullptr;             // per head: dimp key rows, then vdimp value rows (rows past dim / vdim are zero)
+    const int32_t *seq_pos = nullptr, *page_table = nullptr;
+    uint32_t pt_stride = 0, page_size = 0, max_pos = 0;
+    void *cache = nullptr;                    // [slot][rankp + rotp], activation type
+    bool ingest = false;                      // a prompt chunk of one sequence
+    // scratch (sizes: QbLatentScratch)
+    void *q = nullptr, *qa = nullptr;
+    float *part_acc = nullptr, *part_ml = nullptr;
+    QbActBuf lat;
+    __nv_bfloat16 *kr = nullptr, *kv = nullptr;
+    QbActBuf out;                             // [rows][H*vdim]
+    bool f32 = false;
+    __host__ __device__ uint32_t dimp() const { return (dim + 15) & ~15u; }
+    __host__ __device__ uint32_t rotp() const { return (rot_dim + 15) & ~15u; }
+    __host__ __device__ uint32_t vdimp() const { return (vdim + 15) & ~15u; }
+    __host__ __device__ uint32_t rankp() const { return (rank + 15) & ~15u; }
+    __host__ __device__ uint32_t pitch() const { return rankp() + rotp(); }
+};
+static const uint32_t QB_LAT_ABSORB_ROWS = 16;     // rows per sequence up to which the absorbed form runs
+static const uint32_t QB_LAT_SPLIT = 128;          // keys per split of the absorbed form
+// Whether prompt chunks of this shape expand keys and values (bfloat16, sizes within the kernel's registers).
+bool qb_latent_expands(const QbLatent &a);
+// Floats of part_acc for up to `rows_cap` prompt rows / n_seqs decode rows with max_keys keys.
+size_t qb_latent_part_floats(const QbLatent &a, uint32_t rows_cap, uint32_t n_seqs, uint32_t max_keys);
+int qb_launch_latent(qb_ctx *ctx, const QbLatent &a);

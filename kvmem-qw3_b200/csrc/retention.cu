@@ -1,0 +1,326 @@
+// Retention: linear attention with one fixed decay per head, an RMS-normalised and gated output, 32-bit state.
+//
+// Decode rows (retention_step_kernel): one launch takes the projections (adding their K-segment partial sums), rotates q
+// and k, advances the state row by row and writes the gated output.  A CTA owns a slice of a head's value columns; the
+// slices of a head form a thread-block cluster that adds up the head's mean square through distributed shared memory.
+//
+// Prompt chunks (retention_chunk_kernel): blocks of 64 rows.  With D[i][j] = decay^(i-j) below the diagonal,
+//     O = (Q K^T . D) V + diag(decay^(i+1)) Q S        S' = decay^n S + sum_j decay^(n-1-j) k_j v_j^T
+// everything in fp32 on the CUDA cores; powers of the decay come from a table made in double precision.
+#include "layered.h"
+
+#include <cooperative_groups.h>
+namespace cg = cooperative_groups;
+
+namespace {
+
+constexpr int RT = 256;
+constexpr uint32_t C = QB_RET_CHUNK, VCH = 32;
+
+template <typename T>
+__global__ void __launch_bounds__(RT)
+retention_step_kernel(QbRetention a, uint32_t vc) {
+    QB_PDL_ENTER();
+    cg::cluster_group cl = cg::this_cluster();
+    extern __shared__ float sm[];
+    float *st = sm;                               // [dim][vc]
+    float *qs = st + (size_t)a.dim * vc, *ks = qs + a.dim;
+    float *cs = ks + a.dim, *sn = cs + a.rot.dims / 2;
+    float *red = sn + a.rot.dims / 2;             // [8][vc]
+    __shared__ float xch[2][16];
+    const uint32_t tid = threadIdx.x, h = blockIdx.y, s = blockIdx.z, v0 = blockIdx.x * vc;
+    const uint32_t nv = min(vc, a.vdim - v0), rank = cl.block_rank(), csize = cl.num_blocks();
+    const uint32_t rows = a.ns * a.R;
+    const size_t ps = (size_t)rows * a.stride;
+    const float decay = a.powers[h * (C + 1) + 1], kscale = 1.0f / sqrtf((float)a.dim);
+    float *gst = a.state + ((size_t)s * a.H + h) * a.dim * a.vdim + v0;
+    for (uint32_t i = tid; i < a.dim * vc; i += RT) {
+        const uint32_t d = i / vc, c = i % vc;
+        st[i] = c < nv ? gst[(size_t)d * a.vdim + c] : 0.0f;
+    }
+    const uint32_t kb = a.H * a.dim, vb = 2 * kb, gb = vb + a.H * a.vdim;
+    const uint32_t half = a.rot.dims / 2;
+    for (uint32_t r = 0; r < a.R; ++r) {
+        const size_t m = (size_t)s * a.R + r, base = m * a.stride;
+        const int pos = a.seq_pos[s] + (int)r;
+        for (uint32_t i = tid; i < half; i += RT) qb_rot_angle(a.rot, pos, i, cs[i], sn[i]);
+        __syncthreads();
+        for (uint32_t d = tid; d < a.dim; d += RT) {
+            float q = qb_ldsum(a.proj, base + h * a.dim + d, a.S, ps), k = qb_ldsum(a.proj, base + kb + h * a.dim + d, a.S, ps);
+            if (d < a.rot.dims) {
+                uint32_t i, p; bool first;
+                qb_rot_pair(a.rot, d, i, p, first);
+                const float q2 = qb_ldsum(a.proj, base + h * a.dim + p, a.S, ps), k2 = qb_ldsum(a.proj, base + kb + h * a.dim + p, a.S, ps);
+                q = first ? q * cs[i] - q2 * sn[i] : q * cs[i] + q2 * sn[i];
+                k = first ? k * cs[i] - k2 * sn[i] : k * cs[i] + k2 * sn[i];
+            }
+            qs[d] = q;
+            ks[d] = k * kscale;
+        }
+        __syncthreads();
+        const uint32_t rg = tid >> 5;
+        for (uint32_t c = tid & 31; c < vc; c += 32) {
+            const float v = c < nv ? qb_ldsum(a.proj, base + vb + h * a.vdim + v0 + c, a.S, ps) : 0.0f;
+            float o = 0.0f;
+#pragma unroll 4
+            for (uint32_t d = rg; d < a.dim; d += RT / 32) {
+                const float t = fmaf(st[d * vc + c], decay, ks[d] * v);
+                st[d * vc + c] = t;
+                o = fmaf(t, qs[d], o);
+            }
+            red[rg * vc + c] = o;
+        }
+        __syncthreads();
+        if (tid < 32) {
+            float ss = 0.0f;
+            for (uint32_t c = tid; c < vc; c += 32) {
+                float o = 0.0f;
+#pragma unroll
+                for (uint32_t g = 0; g < RT / 32; ++g) o += red[g * vc + c];
+                red[c] = o;
+                ss += o * o;
+            }
+            ss = warp_sum(ss);
+            if (tid < csize) cl.map_shared_rank(&xch[0][0], tid)[(r & 1) * 16 + rank] = ss;
+        }
+        cl.sync();                                   // every slice's sum is here (and red[] within the CTA)
+        float tot = 0.0f;
+        for (uint32_t i = 0; i < csize; ++i) tot += xch[r & 1][i];
+        const float inv = rsqrtf(tot / (float)a.vdim + a.eps);
+        T *out = (T *)a.out.p + m * a.out.ld + h * a.vdim + v0;
+        for (uint32_t c = tid; c < nv; c += RT) {
+            const float g = qb_ldsum(a.proj, base + gb + h * a.vdim + v0 + c, a.S, ps);
+            out[c] = qb_cast<T>(red[c] * inv * qb_swiglu(g, 1.0f));
+        }
+        __syncthreads();
+    }
+    for (uint32_t i = tid; i < a.dim * vc; i += RT) {
+        const uint32_t d = i / vc, c = i % vc;
+        if (c < nv) gst[(size_t)d * a.vdim + c] = st[i];
+    }
+    cl.sync();                                       // no CTA leaves while a peer may still write its xch
+}
+
+// Rotates q and k of a prompt chunk in place (k also scaled); adds K-segment partial sums of every column first.
+__global__ void __launch_bounds__(RT)
+retention_rotate_kernel(QbRetention a) {
+    QB_PDL_ENTER();
+    extern __shared__ float sm[];
+    const uint32_t m = blockIdx.x, half = a.rot.dims / 2, s = m / a.R;
+    float *cs = sm, *sn = sm + half;
+    const int pos = a.seq_pos[s] + (int)(m % a.R);
+    for (uint32_t i = threadIdx.x; i < half; i += RT) qb_rot_angle(a.rot, pos, i, cs[i], sn[i]);
+    __syncthreads();
+    const size_t base = (size_t)m * a.stride, ps = (size_t)a.ns * a.R * a.stride;
+    const float kscale = 1.0f / sqrtf((float)a.dim);
+    float *row = a.proj + base;
+    // rotated pairs
+    for (uint32_t t = threadIdx.x; t < 2 * a.H * half; t += RT) {
+        const uint32_t i = t % half, hh = t / half;                           // hh < H: q heads, then k heads
+        const uint32_t j = hh * a.dim + (a.rot.interleaved ? 2 * i : i), p = a.rot.interleaved ? j + 1 : j + half;
+        const float u = qb_ldsum(a.proj, base + j, a.S, ps), v = qb_ldsum(a.proj, base + p, a.S, ps), sc = hh < a.H ? 1.0f : kscale;
+        row[j] = (u * cs[i] - v * sn[i]) * sc;
+        row[p] = (v * cs[i] + u * sn[i]) * sc;
+    }
+    // dimensions that pass
+    const uint32_t rest = a.dim - a.rot.dims;
+    for (uint32_t t = threadIdx.x; t < 2 * a.H * rest; t += RT) {
+        const uint32_t hh = t / rest, j = hh * a.dim + a.rot.dims + t % rest;
+        row[j] = qb_ldsum(a.proj, base + j, a.S, ps) * (hh < a.H ? 1.0f : kscale);
+    }
+    if (a.S > 1)
+        for (uint32_t j = 2 * a.H * a.dim + threadIdx.x; j < a.stride; j += RT) row[j] = qb_ldsum(a.proj, base + j, a.S, ps);
+}
+
+// grid (value slices, H, sequences).  q and k are rotated and scaled; the outputs replace the v columns of the projection.
+__global__ void __launch_bounds__(RT)
+retention_chunk_kernel(QbRetention a, uint32_t dimr) {
+    QB_PDL_ENTER();
+    extern __shared__ float4 sm4[];
+    float *sm = reinterpret_cast<float *>(sm4);
+    const uint32_t dp = dimr + 4;
+    constexpr uint32_t PP = C + 4;
+    float *qs = sm, *ks = qs + C * dp, *vs = ks + C * dp, *st = vs + C * VCH, *pm = st + dimr * VCH, *pw = pm + C * PP;
+    const uint32_t tid = threadIdx.x, h = blockIdx.y, s = blockIdx.z, v0 = blockIdx.x * VCH;
+    const uint32_t nv = min(VCH, a.vdim - v0);
+    float *gst = a.state + ((size_t)s * a.H + h) * a.dim * a.vdim + v0;
+    for (uint32_t i = tid; i < dimr * VCH; i += RT) {
+        const uint32_t d = i / VCH, c = i % VCH;
+        st[i] = (d < a.dim && c < nv) ? gst[(size_t)d * a.vdim + c] : 0.0f;
+    }
+    for (uint32_t i = tid; i <= C; i += RT) pw[i] = a.powers[h * (C + 1) + i];
+    const uint32_t kb = a.H * a.dim, vb = 2 * kb;
+    for (uint32_t r0 = 0; r0 < a.R; r0 += C) {
+        const uint32_t n = min(C, a.R - r0);
+        float *rows = a.proj + ((size_t)s * a.R + r0) * a.stride;
+        for (uint32_t i = tid; i < C * dimr; i += RT) {
+            const uint32_t r = i / dimr, d = i % dimr;
+            const bool in = r < n && d < a.dim;
+            qs[r * dp + d] = in ? rows[(size_t)r * a.stride + h * a.dim + d] : 0.0f;
+            ks[r * dp + d] = in ? rows[(size_t)r * a.stride + kb + h * a.dim + d] : 0.0f;
+        }
+        for (uint32_t i = tid; i < C * VCH; i += RT) {
+            const uint32_t r = i / VCH, c = i % VCH;
+            vs[i] = (r < n && c < nv) ? rows[(size_t)r * a.stride + vb + h * a.vdim + v0 + c] : 0.0f;
+        }
+        __syncthreads();
+        {   // decayed scores
+            const uint32_t tx = tid & 15, ty = tid >> 4;
+            float acc[4][4] = {};
+            for (uint32_t d = 0; d < dimr; d += 4) {
+                float4 q[4], k[4];
+#pragma unroll
+                for (int i = 0; i < 4; ++i) {
+                    q[i] = *reinterpret_cast<const float4 *>(qs + (ty * 4 + i) * dp + d);
+                    k[i] = *reinterpret_cast<const float4 *>(ks + (tx + 16 * i) * dp + d);
+                }
+#pragma unroll
+                for (int i = 0; i < 4; ++i)
+#pragma unroll
+                    for (int j = 0; j < 4; ++j)
+                        acc[i][j] = fmaf(q[i].x, k[j].x, fmaf(q[i].y, k[j].y, fmaf(q[i].z, k[j].z, fmaf(q[i].w, k[j].w, acc[i][j]))));
+            }
+#pragma unroll
+            for (int i = 0; i < 4; ++i)
+#pragma unroll
+                for (int j = 0; j < 4; ++j) {
+                    const uint32_t ri = ty * 4 + i, cj = tx + 16 * j;
+                    pm[ri * PP + cj] = cj <= ri ? acc[i][j] * pw[ri - cj] : 0.0f;
+                }
+        }
+        __syncthreads();
+        {   // outputs: rows r, r + 32; four columns
+            const uint32_t c = (tid & 7) * 4, r = tid >> 3;
+            float o[2][4] = {};
+            for (uint32_t d = 0; d < dimr; d += 4) {
+                float4 sv[4];
+#pragma unroll
+                for (int i = 0; i < 4; ++i) sv[i] = *reinterpret_cast<const float4 *>(st + (d + i) * VCH + c);
+#pragma unroll
+                for (int k = 0; k < 2; ++k) {
+                    const float4 q = *reinterpret_cast<const float4 *>(qs + (r + 32 * k) * dp + d);
+                    const float qa[4] = {q.x, q.y, q.z, q.w};
+#pragma unroll
+                    for (int i = 0; i < 4; ++i) {
+                        o[k][0] = fmaf(qa[i], sv[i].x, o[k][0]); o[k][1] = fmaf(qa[i], sv[i].y, o[k][1]);
+                        o[k][2] = fmaf(qa[i], sv[i].z, o[k][2]); o[k][3] = fmaf(qa[i], sv[i].w, o[k][3]);
+                    }
+                }
+            }
+#pragma unroll
+            for (int k = 0; k < 2; ++k)
+#pragma unroll
+                for (int i = 0; i < 4; ++i) o[k][i] *= pw[r + 32 * k + 1];
+            for (uint32_t j = 0; j < C; j += 4) {
+                float4 vv[4];
+#pragma unroll
+                for (int i = 0; i < 4; ++i) vv[i] = *reinterpret_cast<const float4 *>(vs + (j + i) * VCH + c);
+#pragma unroll
+                for (int k = 0; k < 2; ++k) {
+                    const float4 p = *reinterpret_cast<const float4 *>(pm + (r + 32 * k) * PP + j);
+                    const float pa[4] = {p.x, p.y, p.z, p.w};
+#pragma unroll
+                    for (int i = 0; i < 4; ++i) {
+                        o[k][0] = fmaf(pa[i], vv[i].x, o[k][0]); o[k][1] = fmaf(pa[i], vv[i].y, o[k][1]);
+                        o[k][2] = fmaf(pa[i], vv[i].z, o[k][2]); o[k][3] = fmaf(pa[i], vv[i].w, o[k][3]);
+                    }
+                }
+            }
+#pragma unroll
+            for (int k = 0; k < 2; ++k)
+#pragma unroll
+                for (int i = 0; i < 4; ++i)
+                    if (r + 32 * k < n && c + i < nv) rows[(size_t)(r + 32 * k) * a.stride + vb + h * a.vdim + v0 + c + i] = o[k][i];
+        }
+        __syncthreads();
+        for (uint32_t t = tid; t < dimr * 2; t += RT) {      // state: four key dims x four columns
+            const uint32_t d = (t >> 3) * 4, c = (t & 7) * 4;
+            float acc[4][4];
+#pragma unroll
+            for (int i = 0; i < 4; ++i)
+#pragma unroll
+                for (int k = 0; k < 4; ++k) acc[i][k] = st[(d + i) * VCH + c + k] * pw[n];
+            for (uint32_t j = 0; j < n; ++j) {
+                const float w = pw[n - 1 - j];
+                float4 v = *reinterpret_cast<const float4 *>(vs + j * VCH + c);
+                const float4 k = *reinterpret_cast<const float4 *>(ks + j * dp + d);
+                v.x *= w; v.y *= w; v.z *= w; v.w *= w;
+                const float ka[4] = {k.x, k.y, k.z, k.w};
+#pragma unroll
+                for (int i = 0; i < 4; ++i) {
+                    acc[i][0] = fmaf(ka[i], v.x, acc[i][0]); acc[i][1] = fmaf(ka[i], v.y, acc[i][1]);
+                    acc[i][2] = fmaf(ka[i], v.z, acc[i][2]); acc[i][3] = fmaf(ka[i], v.w, acc[i][3]);
+                }
+            }
+#pragma unroll
+            for (int i = 0; i < 4; ++i)
+#pragma unroll
+                for (int k = 0; k < 4; ++k) st[(d + i) * VCH + c + k] = acc[i][k];
+        }
+        __syncthreads();
+    }
+    for (uint32_t i = tid; i < a.dim * VCH; i += RT) {
+        const uint32_t d = i / VCH, c = i % VCH;
+        if (c < nv) gst[(size_t)d * a.vdim + c] = st[i];
+    }
+}
+
+// One warp per (row, head): root mean square of the output (in the v columns) and the gate.
+template <typename T>
+__global__ void __launch_bounds__(RT)
+retention_gate_kernel(QbRetention a) {
+    QB_PDL_ENTER();
+    const uint32_t t = blockIdx.x * (RT / 32) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+    if (t >= a.ns * a.R * a.H) return;
+    const uint32_t m = t / a.H, h = t % a.H;
+    const float *o = a.proj + (size_t)m * a.stride + 2 * a.H * a.dim + h * a.vdim, *g = o + a.H * a.vdim;
+    float ss = 0.0f;
+    for (uint32_t c = lane; c < a.vdim; c += 32) ss += o[c] * o[c];
+    const float inv = rsqrtf(warp_sum(ss) / (float)a.vdim + a.eps);
+    T *out = (T *)a.out.p + (size_t)m * a.out.ld + h * a.vdim;
+    for (uint32_t c = lane; c < a.vdim; c += 32) out[c] = qb_cast<T>(o[c] * inv * qb_swiglu(g[c], 1.0f));
+}
+
+template <typename T>
+int launch_step(qb_ctx *ctx, const QbRetention &a) {
+    uint32_t vc = VCH;
+    while ((a.vdim + vc - 1) / vc > 8) vc += VCH;
+    const uint32_t split = (a.vdim + vc - 1) / vc;
+    const size_t smem = ((size_t)a.dim * vc + 2 * a.dim + a.rot.dims + (RT / 32) * vc) * sizeof(float);
+    QB_REQUIRE(smem <= 220 * 1024, "retention: head of %u x %u does not fit", a.dim, a.vdim);
+    QB_CUDA(cudaFuncSetAttribute(retention_step_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    cudaLaunchConfig_t cfg = {};
+    cfg.gridDim = dim3(split, a.H, a.ns);
+    cfg.blockDim = dim3(RT);
+    cfg.dynamicSmemBytes = smem;
+    cfg.stream = ctx->stream;
+    cudaLaunchAttribute attr[2];
+    attr[0].id = cudaLaunchAttributeClusterDimension;
+    attr[0].val.clusterDim.x = split; attr[0].val.clusterDim.y = 1; attr[0].val.clusterDim.z = 1;
+    attr[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    attr[1].val.programmaticStreamSerializationAllowed = 1;
+    cfg.attrs = attr;
+    cfg.numAttrs = 2;
+    QB_CUDA(cudaLaunchKernelEx(&cfg, retention_step_kernel<T>, a, vc));
+    QB_LAUNCHED(ctx, "retention_step_kernel");
+    return QB_OK;
+}
+
+}  // namespace
+
+int qb_launch_retention(qb_ctx *ctx, const QbRetention &a) {
+    QB_REQUIRE(a.ns > 0 && a.R > 0 && a.rot.dims <= a.dim && a.stride == 2 * a.H * (a.dim + a.vdim), "retention: bad arguments");
+    const uint32_t dimr = (a.dim + 3) & ~3u;
+    const size_t smem = ((size_t)2 * C * (dimr + 4) + C * VCH + (size_t)dimr * VCH + C * (C + 4) + C + 1) * sizeof(float);
+    if (a.R < 16 || smem > 220 * 1024) return a.out.f32 ? launch_step<float>(ctx, a) : launch_step<__nv_bfloat16>(ctx, a);
+    QB_CUDA(qb_launch_pdl(ctx->stream, retention_rotate_kernel, dim3(a.ns * a.R), dim3(RT), (size_t)(a.rot.dims * sizeof(float)), a));
+    QB_LAUNCHED(ctx, "retention_rotate_kernel");
+    QB_CUDA(cudaFuncSetAttribute(retention_chunk_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    QB_CUDA(qb_launch_pdl(ctx->stream, retention_chunk_kernel, dim3((a.vdim + VCH - 1) / VCH, a.H, a.ns), dim3(RT), smem, a, dimr));
+    QB_LAUNCHED(ctx, "retention_chunk_kernel");
+    const dim3 grid((a.ns * a.R * a.H + RT / 32 - 1) / (RT / 32));
+    if (a.out.f32) QB_CUDA(qb_launch_pdl(ctx->stream, retention_gate_kernel<float>, grid, dim3(RT), (size_t)0, a));
+    else QB_CUDA(qb_launch_pdl(ctx->stream, retention_gate_kernel<__nv_bfloat16>, grid, dim3(RT), (size_t)0, a));
+    QB_LAUNCHED(ctx, "retention_gate_kernel");
+    return QB_OK;
+}
