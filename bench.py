@@ -23,6 +23,7 @@ Other workloads, one GPU, for profiling (each prints its own lines):
     --workload attn      paged gated attention alone at --ctx (comma list), cold L2
     --workload timeline  per-launch device timeline of the tensor-core GEMMs of one step
     --workload serve     the continuous-batching loops at the 27B shape, wall clock
+    --workload kezilix   prefill and decode of the Kezilix design beside the qwen35 hybrid at equal size, per kernel
     --workload tokenizer the byte-level BPE tokenizer on the host (no GPU): MB/s beside the reference's own, where built
 """
 import argparse
@@ -56,7 +57,7 @@ def parse_args():
     ap.add_argument("--steps", type=int, default=40)
     ap.add_argument("--warmup", type=int, default=4)
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
-    ap.add_argument("--workload", default="step", choices=["step", "gemm", "attn", "timeline", "serve", "tokenizer"])
+    ap.add_argument("--workload", default="step", choices=["step", "gemm", "attn", "timeline", "serve", "kezilix", "tokenizer"])
     ap.add_argument("--sub", default="all", choices=["all", "none"], help="the short runs of configurations 3, 4, 5 / the TP FFN pair")
     ap.add_argument("--layers", type=int, default=64, help="target layers (64 = the 27B-class shape)")
     ap.add_argument("--prompt", type=int, default=PROMPT_LEN)
@@ -71,6 +72,7 @@ def parse_args():
     ap.add_argument("--impls", default="1,2")
     ap.add_argument("--ctx", default="2048,32768")
     ap.add_argument("--tp", action="store_true", help="--workload gemm: the tensor-parallel FFN pair over the ranks of this launch")
+    ap.add_argument("--sizes", default="2048x6144,4096x12288,5120x17408", help="--workload kezilix: width x feed-forward size, comma list")
     ap.add_argument("--slots", type=int, default=8)
     ap.add_argument("--requests", type=int, default=24)
     return ap.parse_args()
@@ -880,6 +882,154 @@ def workload_serve(args):
     model.close(); ctx.close()
 
 
+def bf16_peak():
+    try:
+        return float(json.load(open(os.path.join(ROOT, "MEASURED_PEAKS.json")))["bf16_tflops"])
+    except Exception:
+        return 1590.0
+
+
+FP32_PEAK_TFLOPS = 148 * 128 * 2 * 1.965e-3      # nominal, CUDA cores
+
+
+def family_bounds(family, cfg, rows, keys, ingest):
+    """{kernel group: least microseconds of one forward} from algorithmic bytes / FLOPs and the measured peaks.  rows: tokens
+    per forward; keys: {sequence: context} -> number of keys each decode row attends, or the prompt length (ingest)."""
+    hbm, _ = peaks()
+    us = lambda nbytes, tflop=0.0, peak=1.0: max(nbytes / hbm * 1e-3, tflop / peak * 1e6)
+    out = {"gemm": 0.0, "recurrent": 0.0, "attention": 0.0, "norm": 0.0}
+    if family == "kezilix":
+        D, V, L = cfg["width"], cfg["vocab"], cfg["layers"]
+        ff = L[0]["mlp"]["ff"]
+    else:
+        D, V, ff = cfg.n_embd, cfg.vocab_size, cfg.n_ff
+        L = [{"type": "latent_attention" if (i + 1) % 4 == 0 else "retention"} for i in range(cfg.n_layers)]
+    wb, peak = (2.0, bf16_peak()) if family == "kezilix" else (34.0 / 32.0, INT8_PEAK_TOPS)
+
+    def gemm(N, Kd, m=None):
+        m = m or rows
+        out["gemm"] += us(N * Kd * wb + m * Kd * wb + m * N * 4.0, 2.0 * m * N * Kd * 1e-12, peak)
+    pairs = float(keys) * (keys + 1) / 2 if ingest else float(rows) * keys
+    for l in L:
+        recurrent = l["type"] == "retention"
+        if family == "kezilix":
+            m = l["mixer"]
+            H, d, v = m["heads"], m["dim"], m["vdim"]
+            if recurrent:
+                gemm(2 * H * (d + v), D)
+                st = 2.0 * H * d * v * 4 * (1 if ingest else rows)
+                fl = rows * H * (2.0 * d * v * 2 + (64 * (d + v) if ingest else 0))
+                out["recurrent"] += us(st + rows * 2.0 * H * (d + v) * 4 + rows * H * v * 2, fl * 1e-12, FP32_PEAK_TFLOPS)
+            else:
+                r, k = m["rot_dim"], m["kv_rank"]
+                gemm(H * (d + r) + k + r, D)
+                if ingest:
+                    gemm(H * (d + v), k, keys)
+                    out["attention"] += us(keys * H * (d + r + v) * 2.0 + rows * H * (d + r + v) * 2.0, pairs * H * 2 * (d + r + v) * 1e-12, bf16_peak())
+                else:
+                    out["attention"] += us(rows * keys * (k + r) * 2.0 + H * (d + v) * k * 2.0, pairs * H * 2 * (2 * k + r) * 1e-12, bf16_peak())
+            gemm(D, H * v)
+        else:
+            hd, H, kv = cfg.head_dim, cfg.n_heads, cfg.n_kv_heads
+            if recurrent:
+                h, nk, nv = cfg.ssm_head_dim, cfg.ssm_num_k_heads, cfg.ssm_num_v_heads
+                n_in = (2 * nk + 2 * nv) * h + 2 * nv
+                gemm(n_in, D)
+                out["recurrent"] += us(2.0 * nv * h * h * 4 * (1 if ingest else rows) + rows * n_in * 4.0 + rows * nv * h * 1.125,
+                                       rows * nv * h * h * 6.0 * 1e-12, FP32_PEAK_TFLOPS)
+                gemm(D, nv * h)
+            else:
+                gemm(2 * H * hd + 2 * kv * hd, D)
+                out["attention"] += us((keys if ingest else rows * keys) * kv * hd * 4.0 + rows * H * hd * 5.0, pairs * H * 4 * hd * 1e-12, bf16_peak())
+                gemm(D, H * hd)
+        gemm(2 * ff, D)
+        gemm(D, ff)
+        out["norm"] += 2 * us(rows * D * (4.0 * 3 + 2.0))
+    gemm(V, D, 1 if ingest else rows)
+    return out
+
+
+KERNEL_GROUPS = (("gemm", ("gemm",)), ("recurrent", ("retention", "dn_")), ("attention", ("latent", "attn", "qk_norm")), ("norm", ("norm_quant", "layer_norm")))
+
+
+def kernel_groups(trace):
+    """Microseconds per kernel group, and per kernel, of a launch trace."""
+    out, names = {}, {}
+    for name, n, us in trace:
+        g = next((g for g, keys in KERNEL_GROUPS if any(k in name for k in keys)), "other")
+        out[g] = out.get(g, 0.0) + us
+        names[name] = [n, round(us / n, 2)]
+    return out, names
+
+
+def workload_kezilix(args):
+    """Prefill and decode throughput of the Kezilix design (bfloat16) and of the qwen35 hybrid (Q8_0) at equal width,
+    feed-forward size and depth (seeded random weights), with the time of every kernel group beside its bound: weights and
+    caches exceed L2, 3 warm-up iterations, CUDA events.  The per-kernel times come from a pass with an event after every
+    launch (no overlap between launches, about 2 us each)."""
+    pkg = entry.load_package()
+    ctx = pkg.Context(0)
+    plen = args.prompt
+
+    def timed(fn, n):
+        e0, e1 = ctx.event(), ctx.event()
+        for _ in range(3):
+            fn()
+        ctx.sync()
+        ctx.record(e0)
+        for _ in range(n):
+            fn()
+        ctx.record(e1)
+        ctx.sync()
+        return ctx.elapsed_ms(e0, e1) / n
+
+    for size in args.sizes.split(","):
+        width, ff = map(int, size.split("x"))
+        for family in ("kezilix", "qwen35"):
+            if family == "kezilix":
+                cfg = pkg.configs.kezilix_bench(width, ff)
+                model, vocab = pkg.Model.layered_synth(ctx, cfg, 7), cfg["vocab"]
+            else:
+                cfg = pkg.configs.qwen35_bench(width, ff)
+                model, vocab = pkg.Model(ctx, cfg, 7), cfg.vocab_size
+            prompt = np.random.RandomState(3).randint(0, vocab, plen).astype(np.int32)
+            rec = {"family": family, "width": width, "ff": ff, "layers": 8, "weight_GB": round(model.weight_bytes / 1e9, 3), "prompt": plen}
+            groups = {}
+
+            def traced(label, fn, bounds):
+                ctx.trace_enable(True)
+                fn()
+                g, names = kernel_groups(ctx.trace_summary())
+                ctx.trace_enable(False)
+                groups[label] = {k: {"us": round(g.get(k, 0.0), 1), "bound_us": round(bounds[k], 1), "times_bound": round(g[k] / bounds[k], 2) if bounds[k] and k in g else None}
+                                 for k in bounds}
+                groups[label]["kernels"] = names
+            for ns in (1, 32):
+                b = pkg.Batch(model, ns, plen + 256, 0)
+                if ns == 1:
+                    def ingest():
+                        b.reset(0)
+                        b.prefill(0, prompt)
+                    ms = timed(ingest, args.iters)
+                    rec["prefill_tok_per_s"] = round(plen / ms * 1e3)
+                    rec["prefill_ms"] = round(ms, 3)
+                    traced("prefill", ingest, family_bounds(family, cfg, plen, plen, True))
+                for s in range(ns):
+                    b.reset(s)
+                    b.prefill(s, prompt)
+                b.read_output()
+                ms = timed(b.greedy_step, 40)
+                rec["decode_b%d_tok_per_s" % ns] = round(ns / ms * 1e3, 1)
+                rec["decode_b%d_ms" % ns] = round(ms, 4)
+                b.read_output()
+                traced("decode_b%d" % ns, b.greedy_step, family_bounds(family, cfg, ns, plen + 44, False))
+                b.close()
+            rec["groups"] = groups
+            model.close()
+            print(json.dumps(rec), flush=True)
+    ctx.close()
+
+
 def workload_tokenizer(args):
     """Host only.  A seeded chat-shaped text (about 2 MB) through the product's tokenizer and, as the CPU baseline, through
     the reference's own (oracle/_ref/libqw3ref_tokenizer.so, where it has been built) on the same seeded vocabulary."""
@@ -940,7 +1090,7 @@ def main():
     local_rank = int(os.environ.get("LOCAL_RANK", "0"))
     if args.workload != "step":
         return {"gemm": workload_gemm, "attn": workload_attn, "timeline": workload_timeline, "serve": workload_serve,
-                "tokenizer": workload_tokenizer}[args.workload](args)
+                "kezilix": workload_kezilix, "tokenizer": workload_tokenizer}[args.workload](args)
     if args.impl == "reference":
         run_reference(args, rank)
         return

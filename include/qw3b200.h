@@ -163,6 +163,17 @@ int qb_weight_q8_0_gate_up(qb_ctx *ctx, const void *gate_blocks, const void *up_
 int qb_q8_0_matmul_silu_mul_q8(qb_ctx *ctx, const qb_weight *gate_up, const float *x_dev, uint32_t M, uint32_t x_stride,
                                int8_t *hq_dev, float *hd_dev, int mode);
 
+/* ---- dense bfloat16 products (the layered models; no counterpart in the reference's Q8_0 path) ------------------- */
+
+typedef struct qb_dense qb_dense;
+/* A bfloat16 matrix [rows][cols] in the tensor cores' operand order, from host memory or seeded. */
+int  qb_dense_weight(qb_ctx *ctx, const void *host_bf16, uint32_t rows, uint32_t cols, qb_dense **out);
+int  qb_dense_weight_synth(qb_ctx *ctx, uint64_t seed, uint32_t rows, uint32_t cols, qb_dense **out);
+void qb_dense_weight_free(qb_ctx *ctx, qb_dense *w);
+/* y[m][n] = sum_k w[n][k] x[m][k], fp32 in and out: x rounded to bfloat16 and tcgen05 products with fp32 accumulation, or
+ * (f32 != 0) plain fp32 arithmetic. */
+int  qb_dense_matmul(qb_ctx *ctx, const qb_dense *w, const float *x_dev, uint32_t M, uint32_t x_stride, float *y_dev, int f32);
+
 /* ---- element-wise / norm / rope / embedding --------------------------------------- */
 
 /* q8_get_rows_batch_kernel (src/kernels_cuda.cu:2075-2157): out[i][:] = dequant(row ids[i]). */

@@ -97,6 +97,10 @@ SIGNATURES = {
     "qb_model_create_synth": (i32, [vp, C.POINTER(ModelConfig), u64, C.POINTER(vp)]),
     "qb_model_create": (i32, [vp, C.POINTER(ModelConfig), C.POINTER(TensorDesc), sz, C.POINTER(vp)]),
     "qb_model_load_gguf": (i32, [vp, C.c_char_p, C.POINTER(vp), C.POINTER(ModelConfig)]),
+    "qb_dense_weight": (i32, [vp, vp, u32, u32, C.POINTER(vp)]),
+    "qb_dense_weight_synth": (i32, [vp, u64, u32, u32, C.POINTER(vp)]),
+    "qb_dense_weight_free": (None, [vp, vp]),
+    "qb_dense_matmul": (i32, [vp, vp, vp, u32, u32, vp, i32]),
     "qb_model_load": (i32, [vp, C.c_char_p, i32, C.POINTER(vp), C.POINTER(ModelConfig)]),
     "qb_model_create_layered_synth": (i32, [vp, C.c_char_p, u64, i32, C.POINTER(vp)]),
     "qb_gguf_read_config": (i32, [C.c_char_p, C.POINTER(ModelConfig), C.POINTER(u64), C.POINTER(u64)]),
@@ -415,6 +419,32 @@ class Weight:
             self.free()
         except Exception:
             pass
+
+
+class DenseWeight:
+    """A bfloat16 matrix in device layout (qb_dense)."""
+
+    def __init__(self, ctx, rows, cols, bits=None, seed=0):
+        """bits: uint16 [rows][cols], the bfloat16 patterns; None: seeded random weights."""
+        self.ctx, self.rows, self.cols = ctx, rows, cols
+        h = vp()
+        if bits is None:
+            check(lib().qb_dense_weight_synth(ctx.h, seed, rows, cols, C.byref(h)))
+        else:
+            bits = np.ascontiguousarray(bits, np.uint16).reshape(rows, cols)
+            check(lib().qb_dense_weight(ctx.h, _np_ptr(bits), rows, cols, C.byref(h)))
+        self.h = h
+
+    def matmul(self, x, f32=False):
+        x = np.ascontiguousarray(x, np.float32)
+        xd, yd = self.ctx.array(x), self.ctx.empty((len(x), self.rows), np.float32)
+        check(lib().qb_dense_matmul(self.ctx.h, self.h, xd.ptr, len(x), x.shape[1], yd.ptr, int(f32)))
+        return yd.download()
+
+    def free(self):
+        if self.h:
+            lib().qb_dense_weight_free(self.ctx.h, self.h)
+            self.h = None
 
 
 def act_ld(M):

@@ -392,7 +392,7 @@ int qb_act_alloc(QbActBuf *a, uint32_t rows, uint32_t cols, bool f32) {
 
 uint32_t qb_dense_split(const QbDense &w, uint32_t M, bool f32, uint32_t sms) {
     if (f32 || M > 64) return 1;
-    const uint32_t tiles = w.rows_pad / 128, slots = (M <= 32 ? 2 : 1) * sms;
+    const uint32_t tiles = w.rows_pad / 128, slots = 2 * sms;       // not a function of M: a decode row's bits do not depend on the batch
     return std::max(1u, std::min({slots / tiles, 8u, w.kc / 4}));
 }
 
@@ -432,4 +432,66 @@ int qb_dense_gate_up(qb_ctx *ctx, const QbDense &w, const QbActBuf &x, uint32_t 
                               F, (__nv_bfloat16 *)out.p, out.ld));
     QB_LAUNCHED(ctx, "dense_swiglu_kernel");
     return QB_OK;
+}
+
+// ---- op-level entry points ----------------------------------------------------------------------------------------------
+namespace {
+__global__ void to_bf16_kernel(const float *__restrict__ x, uint32_t stride, uint32_t K, __nv_bfloat16 *__restrict__ out, uint32_t ld) {
+    const uint32_t k = blockIdx.x * blockDim.x + threadIdx.x, m = blockIdx.y;
+    if (k < K) out[(size_t)m * ld + k] = __float2bfloat16(x[(size_t)m * stride + k]);
+}
+}  // namespace
+
+struct qb_dense { QbDense w; };
+
+extern "C" int qb_dense_weight(qb_ctx *ctx, const void *host_bf16, uint32_t rows, uint32_t cols, qb_dense **out) {
+    QB_REQUIRE(ctx && host_bf16 && out, "qb_dense_weight: null argument");
+    QB_CUDA(cudaSetDevice(ctx->device));
+    auto *d = new qb_dense();
+    QbDenseRows r;
+    r.n = r.group = r.stride = rows;
+    int st = qb_dense_alloc(ctx, rows, cols, &d->w);
+    if (st == QB_OK) st = qb_dense_upload(ctx, &d->w, r, (const uint16_t *)host_bf16);
+    if (st != QB_OK) { qb_dense_free(&d->w); delete d; return st; }
+    *out = d;
+    return QB_OK;
+}
+extern "C" int qb_dense_weight_synth(qb_ctx *ctx, uint64_t seed, uint32_t rows, uint32_t cols, qb_dense **out) {
+    QB_REQUIRE(ctx && out, "qb_dense_weight_synth: null argument");
+    QB_CUDA(cudaSetDevice(ctx->device));
+    auto *d = new qb_dense();
+    QbDenseRows r;
+    r.n = r.group = r.stride = rows;
+    int st = qb_dense_alloc(ctx, rows, cols, &d->w);
+    if (st == QB_OK) st = qb_dense_fill_synth(ctx, &d->w, r, seed, 1, 0.02f);
+    if (st != QB_OK) { qb_dense_free(&d->w); delete d; return st; }
+    *out = d;
+    return QB_OK;
+}
+extern "C" void qb_dense_weight_free(qb_ctx *ctx, qb_dense *d) {
+    if (!d) return;
+    cudaStreamSynchronize(ctx->stream);
+    qb_dense_free(&d->w);
+    delete d;
+}
+extern "C" int qb_dense_matmul(qb_ctx *ctx, const qb_dense *d, const float *x, uint32_t M, uint32_t x_stride, float *y, int f32) {
+    QB_REQUIRE(ctx && d && x && y && M > 0 && x_stride >= d->w.cols, "qb_dense_matmul: bad arguments");
+    QB_CUDA(cudaSetDevice(ctx->device));
+    const QbDense &w = d->w;
+    QbActBuf a;
+    a.cap = M;
+    if (f32) {
+        a.p = const_cast<float *>(x); a.ld = x_stride; a.f32 = true;
+        return qb_dense_gemm(ctx, w, a, M, y, 1);
+    }
+    const uint32_t S = qb_dense_split(w, M, false, (uint32_t)ctx->sm_count);
+    a.ld = (w.cols + 63) / 64 * 64;
+    QB_TRY(qb_ctx_scratch2(ctx, (size_t)M * a.ld * 2, &a.p));
+    to_bf16_kernel<<<dim3((w.cols + 255) / 256, M), 256, 0, ctx->stream>>>(x, x_stride, w.cols, (__nv_bfloat16 *)a.p, a.ld);
+    QB_LAUNCHED(ctx, "to_bf16_kernel");
+    if (S == 1) return qb_dense_gemm(ctx, w, a, M, y, 1);
+    void *parts = nullptr;
+    QB_TRY(qb_ctx_scratch(ctx, (size_t)S * M * w.rows * sizeof(float), &parts));
+    QB_TRY(qb_dense_gemm(ctx, w, a, M, (float *)parts, S));
+    return qb_launch_reduce_parts(ctx, (const float *)parts, S, M, w.rows, y, w.rows);
 }

@@ -8,8 +8,8 @@ slots (an idle slot decodes from its reset state and is reset again before it ru
 result never depends on which other rows share a launch, a request's tokens are the ones it would get alone.
 
 `engine` is anything with n_seqs, k, max_ctx, prefill(seq, tokens, more=False), prefill_sampled(seq, tokens, u, **sampling),
-mtp_step() / mtp_step_sampled(u, **sampling) or greedy_step(), read_output(), reset(seq):
-binding.Batch on the GPU, a fake in the CPU tests.
+mtp_step() / mtp_step_sampled(u, **sampling) for speculative decoding, greedy_step() / sampled_step(u, **sampling) for plain
+steps (models without a draft layer), read_output(), reset(seq): binding.Batch on the GPU, a fake in the CPU tests.
 """
 import collections
 
@@ -93,6 +93,19 @@ class DrawQueue:
         return v
 
 
+def decode_step(engine, speculative, sampling, u):
+    """One decode step of the batch; u: the draws of every slot (sampling only), [n_seqs][per_step]."""
+    if sampling is not None:
+        if speculative:
+            engine.mtp_step_sampled(u, **sampling)
+        else:
+            engine.sampled_step([d[0] for d in u], **sampling)
+    elif speculative:
+        engine.mtp_step()
+    else:
+        engine.greedy_step()
+
+
 class PrefixCache:
     """Host policy over the engine's shared-prefix entries (prefix_capture / prefix_attach / prefix_release), the role of the
     reference server's prefix cache (src/qwen_native_backend.cpp:9785-10410): a prompt is looked up by its page-aligned
@@ -164,8 +177,6 @@ def run_compact(engine, requests, speculative=True, max_steps=1 << 30, sampling=
     pending = collections.deque(sorted(requests, key=lambda r: (r.arrival_step, r.rid)))
     per_step = engine.k + 1 if speculative else 1
     if sampling is not None:
-        if not speculative:
-            raise ValueError("sampled decode runs through the speculative step")
         sampling = dict(sampling)
         presence, repetition = sampling.pop("presence", 0.0), sampling.pop("repetition", 1.0)
         if presence != 0.0 or repetition != 1.0:
@@ -263,13 +274,10 @@ def run_compact(engine, requests, speculative=True, max_steps=1 << 30, sampling=
         if not live:
             step += 1
             continue
+        u = None
         if sampling is not None:
             u = [draws[live[s].rid].peek() if s < len(live) else [0.5] * per_step for s in range(engine.n_seqs)]
-            engine.mtp_step_sampled(u, **sampling)
-        elif speculative:
-            engine.mtp_step()
-        else:
-            engine.greedy_step()
+        decode_step(engine, speculative, sampling, u)
         out = engine.read_output()
         step += 1
         for s in range(len(live) - 1, -1, -1):           # from the end: retiring swaps the last live request in
@@ -293,8 +301,6 @@ def run(engine, requests, speculative=True, max_steps=1 << 30, sampling=None, rn
         sched.submit(r)
     per_step = engine.k + 1 if speculative else 1
     idle_pos = [0] * engine.n_seqs                       # upper bound of the position of slots that hold no request
-    if sampling is not None and not speculative:
-        raise ValueError("sampled decode runs through the speculative step")
     draws = {}                                           # slot -> DrawQueue of the request it holds
     if sampling is not None:
         sampling = dict(sampling)
@@ -324,13 +330,10 @@ def run(engine, requests, speculative=True, max_steps=1 << 30, sampling=None, rn
             if s not in sched.active and idle_pos[s] + 2 * per_step >= engine.max_ctx:
                 engine.reset(s)
                 idle_pos[s] = 0
+        u = None
         if sampling is not None:
             u = [draws[s].peek() if s in sched.active else [0.5] * per_step for s in range(engine.n_seqs)]
-            engine.mtp_step_sampled(u, **sampling)
-        elif speculative:
-            engine.mtp_step()
-        else:
-            engine.greedy_step()
+        decode_step(engine, speculative, sampling, u)
         out = engine.read_output()
         step += 1
         for s in range(engine.n_seqs):
