@@ -18,14 +18,6 @@
 namespace {
 using namespace qbtc;
 
-__device__ __forceinline__ void tc_mma_bf16(uint32_t d_tmem, uint64_t a_desc, uint64_t b_desc, uint32_t idesc, uint32_t accumulate) {
-    asm volatile(
-        "{\n\t.reg .pred p;\n\t"
-        "setp.ne.b32 p, %4, 0;\n\t"
-        "tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, {%5, %6, %7, %8}, p;\n\t}"
-        ::"r"(d_tmem), "l"(a_desc), "l"(b_desc), "r"(idesc), "r"(accumulate), "r"(0u), "r"(0u), "r"(0u), "r"(0u) : "memory");
-}
-
 enum Epi { EPI_PARTS = 0, EPI_BF16 = 1, EPI_SWIGLU = 2 };
 
 template <int NT>
@@ -135,7 +127,7 @@ dense_gemm_kernel(const uint8_t *__restrict__ rec, const __grid_constant__ CUten
                     const uint32_t a_addr = smem_u32(smem + (size_t)st * C::STAGE), b_addr = a_addr + QB_DREC_BYTES;
 #pragma unroll
                     for (int ks = 0; ks < 4; ++ks)
-                        tc_mma_bf16(tmem_base + ab * NT, smem_desc_sw128(a_addr + ks * 32), smem_desc_sw128(b_addr + ks * 32), idesc,
+                        tc_mma_f16(tmem_base + ab * NT, smem_desc_sw128(a_addr + ks * 32), smem_desc_sw128(b_addr + ks * 32), idesc,
                                     (it > 0 || ks > 0) ? 1u : 0u);
                     tc_commit(bar_empty + 8 * st);
                 }
@@ -382,11 +374,11 @@ int qb_dense_fill_synth(qb_ctx *ctx, QbDense *w, const QbDenseRows &rows, uint64
     return QB_OK;
 }
 
-int qb_act_alloc(QbActBuf *a, uint32_t rows, uint32_t cols, bool f32) {
+int qb_act_alloc(qb_ctx *ctx, QbActBuf *a, uint32_t rows, uint32_t cols, bool f32) {
     a->cap = rows; a->ld = (cols + 63) / 64 * 64; a->f32 = f32;
     const size_t bytes = (size_t)rows * a->ld * (f32 ? 4 : 2);
     QB_CUDA(cudaMalloc(&a->p, bytes));
-    QB_CUDA(cudaMemset(a->p, 0, bytes));
+    QB_CUDA(cudaMemsetAsync(a->p, 0, bytes, ctx->stream));
     return QB_OK;
 }
 

@@ -36,7 +36,7 @@ struct QbActBuf {
     uint32_t cap = 0, ld = 0;        // ld in elements, a multiple of 8
     bool f32 = false;
 };
-int qb_act_alloc(QbActBuf *a, uint32_t rows, uint32_t cols, bool f32);
+int qb_act_alloc(qb_ctx *ctx, QbActBuf *a, uint32_t rows, uint32_t cols, bool f32);
 
 // Feed-forward input weight: gate and up rows interleaved in groups of 16 (32 consecutive rows = 16 gate, 16 up).
 __host__ __device__ inline uint32_t qb_gate_col(uint32_t f) { return (f >> 4) * 32 + (f & 15); }

@@ -151,5 +151,4 @@ struct qb_batch {
     uint32_t steps_since_probe = 0;
 };
 
-uint32_t qb_env_u32(const char *name, uint32_t dflt);
 int qb_upload_f32(qb_ctx *ctx, const std::vector<float> &v, float **out);

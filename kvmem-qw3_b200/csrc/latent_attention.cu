@@ -4,9 +4,9 @@
 //
 // Few rows per sequence (decode), and every row in fp32: the absorbed form.  q_n . (W_uk c) = (W_uk^T q_n) . c, so the key
 // projection is applied to the query once (latent_absorb_kernel), all heads of all rows of a sequence then attend the same
-// cached vectors (latent_split_kernel: 16 or 32 (row, head) queries per CTA over a fixed span of keys, mma.sync bf16, the
-// tile of latents serving as keys and as values; latent_split_simt_kernel: the same in fp32), and latent_merge_kernel folds
-// the spans, adds the sink and applies W_uv head by head.
+// cached vectors over spans of keys (latent_split_tc_kernel, latent_attention_tc.cu; shapes it does not take:
+// latent_split_kernel, 16 or 32 (row, head) queries per CTA on mma.sync, the tile of latents serving as keys and as values;
+// latent_split_simt_kernel: the same in fp32), and latent_merge_kernel folds the spans, adds the sink and applies W_uv head by head.
 //
 // Prompt chunks in bfloat16: the latents of all keys are gathered from their pages, expanded to keys and values by one
 // GEMM, and latent_prefill_kernel runs a tiled attention per head (128 or 64 rows per CTA, running maximum and sum).
@@ -20,9 +20,10 @@ constexpr int LT = 256;
 constexpr float LOG2E = 1.4426950408889634f;
 
 // ---- new rows: rotate the query, normalise the latent, append to the paged cache ----------------------------------------
+// grid (rows, 1 + head groups): block y = 0 takes the latent and the shared key part, y > 0 `hpb` query heads.
 template <typename T>
 __global__ void __launch_bounds__(LT)
-latent_prepare_kernel(QbLatent a, int *err_flag) {
+latent_prepare_kernel(QbLatent a, uint32_t hpb) {
     QB_PDL_ENTER();
     extern __shared__ float sm[];
     __shared__ float red[LT / 32];
@@ -32,51 +33,61 @@ latent_prepare_kernel(QbLatent a, int *err_flag) {
     const size_t base = (size_t)m * a.stride, ps = (size_t)a.ns * a.R * a.stride;
     const uint32_t hq = a.dim + a.rot_dim, c0 = a.H * hq, k0 = c0 + a.rank;
     for (uint32_t i = tid; i < half; i += LT) qb_rot_angle(a.rot, pos, i, cs[i], sn[i]);
+    auto rotated = [&](uint32_t at, uint32_t j) -> float {          // element j of the rotated vector that starts at column `at`
+        const float v = qb_sum8(a.proj, base + at + j, a.S, ps);
+        if (j >= a.rot.dims) return v;
+        uint32_t i, p; bool first;
+        qb_rot_pair(a.rot, j, i, p, first);
+        const float w = qb_sum8(a.proj, base + at + p, a.S, ps);
+        return first ? v * cs[i] - w * sn[i] : v * cs[i] + w * sn[i];
+    };
+    if (blockIdx.y > 0) {
+        __syncthreads();
+        const uint32_t h0 = (blockIdx.y - 1) * hpb, nh = min(hpb, a.H - h0);
+        const uint32_t dp = a.dimp(), per = dp + a.rotp();
+        T *q = (T *)a.q + ((size_t)m * a.H + h0) * per;
+#pragma unroll 4
+        for (uint32_t i = tid; i < nh * per; i += LT) {
+            const uint32_t h = h0 + i / per, e = i % per;
+            float v = 0.0f;
+            if (e < a.dim) v = qb_sum8(a.proj, base + h * hq + e, a.S, ps);
+            else if (e >= dp && e - dp < a.rot_dim) v = rotated(h * hq + a.dim, e - dp);
+            q[i] = qb_cast<T>(v);
+        }
+        return;
+    }
     float ss = 0.0f;
     for (uint32_t i = tid; i < a.rank; i += LT) {
-        const float v = qb_ldsum(a.proj, base + c0 + i, a.S, ps);
+        const float v = qb_sum8(a.proj, base + c0 + i, a.S, ps);
         lat[i] = v;
         ss += v * v;
     }
     const float inv = rsqrtf(qb_block_sum(ss, red, LT / 32) / (float)a.rank + a.eps);
-    auto rotated = [&](uint32_t at, uint32_t j) -> float {          // element j of the rotated vector that starts at column `at`
-        const float v = qb_ldsum(a.proj, base + at + j, a.S, ps);
-        if (j >= a.rot.dims) return v;
-        uint32_t i, p; bool first;
-        qb_rot_pair(a.rot, j, i, p, first);
-        const float w = qb_ldsum(a.proj, base + at + p, a.S, ps);
-        return first ? v * cs[i] - w * sn[i] : v * cs[i] + w * sn[i];
-    };
     const int32_t page = a.page_table[(size_t)s * a.pt_stride + (uint32_t)pos / a.page_size];
     if (page < 0) {
-        if (tid == 0) atomicExch(err_flag, 3002);                    // an unassigned page: nothing is appended
-    } else {
-        T *slot = (T *)a.cache + ((size_t)page * a.page_size + (uint32_t)pos % a.page_size) * a.pitch();
-        const uint32_t rp = a.rankp();
-        for (uint32_t i = tid; i < a.pitch(); i += LT) {
-            float v = 0.0f;
-            if (i < a.rank) v = lat[i] * inv * a.norm_w[i];
-            else if (i >= rp && i - rp < a.rot_dim) v = rotated(k0, i - rp);
-            slot[i] = qb_cast<T>(v);
-        }
+        if (tid == 0) atomicExch(a.err_flag, 3002);                    // an unassigned page: nothing is appended
+        return;
     }
-    const uint32_t dp = a.dimp(), per = dp + a.rotp();
-    T *q = (T *)a.q + (size_t)m * a.H * per;
-    for (uint32_t i = tid; i < a.H * per; i += LT) {
-        const uint32_t h = i / per, e = i % per;
+    T *slot = (T *)a.cache + ((size_t)page * a.page_size + (uint32_t)pos % a.page_size) * a.pitch();
+    const uint32_t rp = a.rankp();
+    for (uint32_t i = tid; i < a.pitch(); i += LT) {
         float v = 0.0f;
-        if (e < a.dim) v = qb_ldsum(a.proj, base + h * hq + e, a.S, ps);
-        else if (e >= dp && e - dp < a.rot_dim) v = rotated(h * hq + a.dim, e - dp);
-        q[i] = qb_cast<T>(v);
+        if (i < a.rank) v = lat[i] * inv * a.norm_w[i];
+        else if (i >= rp && i - rp < a.rot_dim) v = rotated(k0, i - rp);
+        slot[i] = qb_cast<T>(v);
     }
 }
 
 // ---- absorbed query: qa[row][h] = [W_uk(h)^T q_n | q_r] --------------------------------------------------------------------
-constexpr int AB_ROWS = 8;
-template <typename T>
+// A CTA takes one head, 128 latent columns and AB_ROWS rows; its weights are requested into L2 before it waits for the query.
+template <typename T, int AB_ROWS>
 __global__ void __launch_bounds__(128)
 latent_absorb_kernel(QbLatent a, const uint8_t *__restrict__ rec, uint32_t kc, uint32_t rows) {
-    QB_PDL_ENTER();
+    asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
+    for (uint32_t i = threadIdx.x; i < 2 * a.dim; i += 128)           // two 128-byte lines per weight row
+        if (blockIdx.y * 2 + (i & 1) < kc)
+            asm volatile("prefetch.global.L2 [%0];" ::"l"(rec + qb_dense_offset(kc, blockIdx.x * (a.dimp() + a.vdimp()) + (i >> 1), (blockIdx.y * 2 + (i & 1)) * 8)));
+    asm volatile("griddepcontrol.wait;" ::: "memory");
     extern __shared__ float sm[];
     const uint32_t h = blockIdx.x, row0 = blockIdx.z * AB_ROWS, tid = threadIdx.x;
     const uint32_t nr = min((uint32_t)AB_ROWS, rows - row0);
@@ -92,7 +103,7 @@ latent_absorb_kernel(QbLatent a, const uint8_t *__restrict__ rec, uint32_t kc, u
     float acc[AB_ROWS][8] = {};
     if (c8 < kc * 8) {
         const uint32_t wr0 = h * (dp + a.vdimp());
-#pragma unroll 2
+#pragma unroll(AB_ROWS == 1 ? 8 : 4)
         for (uint32_t d = dg; d < a.dim; d += 8) {
             const uint4 raw = *reinterpret_cast<const uint4 *>(rec + qb_dense_offset(kc, wr0 + d, c8));
             const __nv_bfloat162 *b = reinterpret_cast<const __nv_bfloat162 *>(&raw);
@@ -129,13 +140,14 @@ latent_absorb_kernel(QbLatent a, const uint8_t *__restrict__ rec, uint32_t kc, u
 constexpr int SQ = 8, SK = 32, SCOLS = 4;                             // value columns per thread: up to 4 x 256
 template <typename T>
 __global__ void __launch_bounds__(LT)
-latent_split_simt_kernel(QbLatent a, uint32_t span, uint32_t n_splits) {
+latent_split_simt_kernel(QbLatent a, uint32_t n_splits) {
     QB_PDL_ENTER();
     extern __shared__ float sm[];
     const uint32_t D = a.pitch(), DP = D + 1, tid = threadIdx.x, w = tid >> 5, lane = tid & 31;
     float *qs = sm, *ts = qs + SQ * D, *pr = ts + SK * DP, *al = pr + SQ * SK;
     const uint32_t split = blockIdx.x, s = blockIdx.z, nq = a.R * a.H, q0 = blockIdx.y * SQ;
     const int base = a.seq_pos[s];
+    const uint32_t span = qb_latent_span((uint32_t)base + a.R, a.max_splits);
     const uint32_t q_last = min(q0 + SQ, nq) - 1;
     const int k_begin = (int)(split * span), k_end = min(k_begin + (int)span, base + (int)(q_last / a.H) + 1);
     if (k_begin >= k_end) return;
@@ -240,7 +252,7 @@ __host__ __device__ inline SplitSmem split_smem(uint32_t D, uint32_t MT) {
 }
 template <int MT, int NV>
 __global__ void __launch_bounds__(LT)
-latent_split_kernel(QbLatent a, uint32_t span, uint32_t n_splits) {
+latent_split_kernel(QbLatent a, uint32_t n_splits) {
     QB_PDL_ENTER();
     extern __shared__ __align__(16) uint8_t smem[];
     const uint32_t D = a.pitch(), pitch = (D + 8) * 2, tid = threadIdx.x, w = tid >> 5, lane = tid & 31;
@@ -249,6 +261,7 @@ latent_split_kernel(QbLatent a, uint32_t span, uint32_t n_splits) {
     __nv_bfloat16 *psm = reinterpret_cast<__nv_bfloat16 *>(smem + L.p);
     const uint32_t split = blockIdx.x, s = blockIdx.z, nq = a.R * a.H, q0 = blockIdx.y * 16 * MT;
     const int base = a.seq_pos[s];
+    const uint32_t span = qb_latent_span((uint32_t)base + a.R, a.max_splits);
     const uint32_t q_last = min(q0 + 16 * MT, nq) - 1;
     const int k_begin = (int)(split * span), k_end = min(k_begin + (int)span, base + (int)(q_last / a.H) + 1);
     if (k_begin >= k_end) return;
@@ -382,47 +395,78 @@ latent_split_kernel(QbLatent a, uint32_t span, uint32_t n_splits) {
         }
 }
 
-// ---- fold the spans, add the sink, apply W_uv: grid (H, rows, slices of the value dimensions) ---------------------------------
-template <typename T>
+// ---- fold the spans, add the sink, apply W_uv: grid (H, rows / MB, slices of the value dimensions) ----------------------------
+template <typename T, int MB>
 __global__ void __launch_bounds__(LT)
-latent_merge_kernel(QbLatent a, const uint8_t *__restrict__ rec, uint32_t kc, uint32_t span, uint32_t n_splits) {
-    QB_PDL_ENTER();
+latent_merge_kernel(QbLatent a, const uint8_t *__restrict__ rec, uint32_t kc, uint32_t rows, uint32_t n_splits) {
+    asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
     extern __shared__ float sm[];
-    const uint32_t h = blockIdx.x, m = blockIdx.y, tid = threadIdx.x, w = tid >> 5, lane = tid & 31;
-    const int pos = a.seq_pos[m / a.R] + (int)(m % a.R);
-    const uint32_t n = min((uint32_t)pos / span + 1, n_splits);
-    float *wt = sm, *lat = sm + ((n_splits + 3) & ~3u);                // weights of the spans, the merged latent (kc * 64)
-    const size_t p0 = ((size_t)m * a.H + h) * n_splits;
-    const float *ml = a.part_ml + p0 * 2;
-    const float sink = a.sink[h];
-    float mx = sink;
-    for (uint32_t i = 0; i < n; ++i) mx = fmaxf(mx, ml[2 * i]);
-    float den = expf(sink - mx);
-    for (uint32_t i = 0; i < n; ++i) den += ml[2 * i + 1] * expf(ml[2 * i] - mx);
-    for (uint32_t i = tid; i < n; i += LT) wt[i] = expf(ml[2 * i] - mx) / den;
-    __syncthreads();
-    for (uint32_t c = tid; c < kc * 64; c += LT) {
-        float v = 0.0f;
-        if (c < a.rank)
-            for (uint32_t i = 0; i < n; ++i) v = fmaf(wt[i], a.part_acc[(p0 + i) * a.rank + c], v);
-        lat[c] = v;
-    }
-    __syncthreads();
+    const uint32_t h = blockIdx.x, m0 = blockIdx.y * MB, tid = threadIdx.x, w = tid >> 5, lane = tid & 31;
     const uint32_t per = (a.vdim + gridDim.z - 1) / gridDim.z, v0 = blockIdx.z * per, v1 = min(a.vdim, v0 + per);
     const uint32_t wr0 = h * (a.dimp() + a.vdimp()) + a.dimp();
-    T *out = (T *)a.out.p + (size_t)m * a.out.ld + h * a.vdim;
-    for (uint32_t v = v0 + w; v < v1; v += LT / 32) {
-        float acc = 0.0f;
-        for (uint32_t c8 = lane; c8 < kc * 8; c8 += 32) {
-            const uint4 raw = *reinterpret_cast<const uint4 *>(rec + qb_dense_offset(kc, wr0 + v, c8));
-            const __nv_bfloat162 *b = reinterpret_cast<const __nv_bfloat162 *>(&raw);
-            const float4 l0 = *reinterpret_cast<const float4 *>(lat + c8 * 8), l1 = *reinterpret_cast<const float4 *>(lat + c8 * 8 + 4);
-            const float2 f0 = __bfloat1622float2(b[0]), f1 = __bfloat1622float2(b[1]), f2 = __bfloat1622float2(b[2]), f3 = __bfloat1622float2(b[3]);
-            acc = fmaf(f0.x, l0.x, fmaf(f0.y, l0.y, fmaf(f1.x, l0.z, fmaf(f1.y, l0.w, acc))));
-            acc = fmaf(f2.x, l1.x, fmaf(f2.y, l1.y, fmaf(f3.x, l1.z, fmaf(f3.y, l1.w, acc))));
+    for (uint32_t i = tid; v0 < v1 && i < (v1 - v0) * kc; i += LT)     // this CTA's weights, into L2 while the spans are still computed
+        asm volatile("prefetch.global.L2 [%0];" ::"l"(rec + qb_dense_offset(kc, wr0 + v0 + i / kc, (i % kc) * 8)));
+    asm volatile("griddepcontrol.wait;" ::: "memory");
+    float *wt = sm, *lat = sm + ((MB * n_splits + 3) & ~3u);            // weights of the spans, the merged latents [MB][kc * 64]
+    __shared__ uint32_t cnt[MB];
+    if (w < MB) {
+        const uint32_t m = m0 + w;
+        uint32_t n = 0;
+        if (m < rows) {
+            const uint32_t base = (uint32_t)a.seq_pos[m / a.R], pos = base + m % a.R;
+            n = min(pos / qb_latent_span(base + a.R, a.max_splits) + 1, n_splits);
+            const float *ml = a.part_ml + ((size_t)m * a.H + h) * n_splits * 2;
+            const float sink = a.sink[h];
+            float mx = sink;
+            for (uint32_t i = lane; i < n; i += 32) mx = fmaxf(mx, ml[2 * i]);
+            mx = warp_max(mx);
+            float den = 0.0f;
+            for (uint32_t i = lane; i < n; i += 32) den += ml[2 * i + 1] * expf(ml[2 * i] - mx);
+            den = warp_sum(den) + expf(sink - mx);
+            for (uint32_t i = lane; i < n; i += 32) wt[w * n_splits + i] = expf(ml[2 * i] - mx) / den;
         }
-        acc = warp_sum(acc);
-        if (lane == 0) out[v] = qb_cast<T>(acc);
+        if (lane == 0) cnt[w] = n;
+    }
+    __syncthreads();
+#pragma unroll 2
+    for (uint32_t t = tid; t < MB * kc * 64; t += LT) {
+        const uint32_t r = t / (kc * 64), c = t % (kc * 64), n = cnt[r];
+        float v = 0.0f;
+        if (c < a.rank) {
+            const float *acc = a.part_acc + ((size_t)(m0 + r) * a.H + h) * n_splits * a.rank + c;
+#pragma unroll 8
+            for (uint32_t i = 0; i < n; ++i) v = fmaf(wt[r * n_splits + i], acc[(size_t)i * a.rank], v);
+        }
+        lat[t] = v;
+    }
+    __syncthreads();
+    // four value dimensions per warp at a time: their weights are in flight together and share the reads of the latents
+    constexpr int NVW = 4;
+    for (uint32_t v = v0 + w * NVW; v < v1; v += LT / 32 * NVW) {
+        float acc[NVW][MB] = {};
+        for (uint32_t c8 = lane; c8 < kc * 8; c8 += 32) {
+            uint4 raw[NVW];
+#pragma unroll
+            for (int j = 0; j < NVW; ++j) raw[j] = *reinterpret_cast<const uint4 *>(rec + qb_dense_offset(kc, wr0 + min(v + j, v1 - 1), c8));
+#pragma unroll
+            for (int r = 0; r < MB; ++r) {
+                const float4 l0 = *reinterpret_cast<const float4 *>(lat + r * kc * 64 + c8 * 8), l1 = *reinterpret_cast<const float4 *>(lat + r * kc * 64 + c8 * 8 + 4);
+#pragma unroll
+                for (int j = 0; j < NVW; ++j) {
+                    const __nv_bfloat162 *b = reinterpret_cast<const __nv_bfloat162 *>(&raw[j]);
+                    const float2 f0 = __bfloat1622float2(b[0]), f1 = __bfloat1622float2(b[1]), f2 = __bfloat1622float2(b[2]), f3 = __bfloat1622float2(b[3]);
+                    acc[j][r] = fmaf(f0.x, l0.x, fmaf(f0.y, l0.y, fmaf(f1.x, l0.z, fmaf(f1.y, l0.w, acc[j][r]))));
+                    acc[j][r] = fmaf(f2.x, l1.x, fmaf(f2.y, l1.y, fmaf(f3.x, l1.z, fmaf(f3.y, l1.w, acc[j][r]))));
+                }
+            }
+        }
+#pragma unroll
+        for (int j = 0; j < NVW; ++j)
+#pragma unroll
+            for (int r = 0; r < MB; ++r) {
+                const float t = warp_sum(acc[j][r]);
+                if (lane == 0 && v + j < v1 && m0 + r < rows) ((T *)a.out.p + (size_t)(m0 + r) * a.out.ld + h * a.vdim)[v + j] = qb_cast<T>(t);
+            }
     }
 }
 
@@ -591,76 +635,100 @@ int launch_prefill(qb_ctx *ctx, const QbLatent &a) {
 }
 
 template <int MT, int NV>
-int launch_split(qb_ctx *ctx, const QbLatent &a, uint32_t span, uint32_t n_splits) {
+int launch_split(qb_ctx *ctx, const QbLatent &a, uint32_t n_splits) {
     const size_t smem = split_smem(a.pitch(), MT).total;
     QB_CUDA(cudaFuncSetAttribute(latent_split_kernel<MT, NV>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-    QB_CUDA(qb_launch_pdl(ctx->stream, latent_split_kernel<MT, NV>, dim3(n_splits, (a.R * a.H + 16 * MT - 1) / (16 * MT), a.ns), dim3(LT), smem, a, span, n_splits));
+    QB_CUDA(qb_launch_pdl(ctx->stream, latent_split_kernel<MT, NV>, dim3(n_splits, (a.R * a.H + 16 * MT - 1) / (16 * MT), a.ns), dim3(LT), smem, a, n_splits));
     QB_LAUNCHED(ctx, "latent_split_kernel");
     return QB_OK;
 }
 template <int MT>
-int launch_split_nv(qb_ctx *ctx, const QbLatent &a, uint32_t span, uint32_t n_splits) {
-    if (a.rankp() <= 128) return launch_split<MT, 2>(ctx, a, span, n_splits);
-    if (a.rankp() <= 256) return launch_split<MT, 4>(ctx, a, span, n_splits);
-    return launch_split<MT, 8>(ctx, a, span, n_splits);
+int launch_split_nv(qb_ctx *ctx, const QbLatent &a, uint32_t n_splits) {
+    if (a.rankp() <= 128) return launch_split<MT, 2>(ctx, a, n_splits);
+    if (a.rankp() <= 256) return launch_split<MT, 4>(ctx, a, n_splits);
+    return launch_split<MT, 8>(ctx, a, n_splits);
 }
 template <typename T>
-int launch_simt(qb_ctx *ctx, const QbLatent &a, uint32_t span, uint32_t n_splits) {
+int launch_simt(qb_ctx *ctx, const QbLatent &a, uint32_t n_splits) {
     const uint32_t D = a.pitch();
     const size_t smem = ((size_t)SQ * D + SK * (D + 1) + SQ * SK + SQ) * sizeof(float);
     QB_REQUIRE(smem <= 227 * 1024 && a.rank <= SCOLS * LT, "latent attention: a latent of %u + %u does not fit", a.rank, a.rot_dim);
     QB_CUDA(cudaFuncSetAttribute(latent_split_simt_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-    QB_CUDA(qb_launch_pdl(ctx->stream, latent_split_simt_kernel<T>, dim3(n_splits, (a.R * a.H + SQ - 1) / SQ, a.ns), dim3(LT), smem, a, span, n_splits));
+    QB_CUDA(qb_launch_pdl(ctx->stream, latent_split_simt_kernel<T>, dim3(n_splits, (a.R * a.H + SQ - 1) / SQ, a.ns), dim3(LT), smem, a, n_splits));
     QB_LAUNCHED(ctx, "latent_split_simt_kernel");
     return QB_OK;
 }
 
-template <typename T>
-int latent_absorbed(qb_ctx *ctx, const QbLatent &a) {
-    const uint32_t rows = a.ns * a.R, kc = a.ukv->kc;
-    const size_t sm_a = ((size_t)AB_ROWS * a.dim + 8 * AB_ROWS * 128) * sizeof(float);
-    QB_REQUIRE(sm_a <= 227 * 1024, "latent attention: %u query dimensions do not fit", a.dim);
-    QB_CUDA(cudaFuncSetAttribute(latent_absorb_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sm_a));
-    QB_CUDA(qb_launch_pdl(ctx->stream, latent_absorb_kernel<T>, dim3(a.H, (a.rankp() + 127) / 128, (rows + AB_ROWS - 1) / AB_ROWS), dim3(128), sm_a, a,
-                          (const uint8_t *)a.ukv->rec, kc, rows));
+template <typename T, int AB>
+int launch_absorb(qb_ctx *ctx, const QbLatent &a, uint32_t rows) {
+    const size_t smem = ((size_t)AB * a.dim + 8 * AB * 128) * sizeof(float);
+    QB_REQUIRE(smem <= 227 * 1024, "latent attention: %u query dimensions do not fit", a.dim);
+    QB_CUDA(cudaFuncSetAttribute(latent_absorb_kernel<T, AB>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    QB_CUDA(qb_launch_pdl(ctx->stream, latent_absorb_kernel<T, AB>, dim3(a.H, (a.rankp() + 127) / 128, (rows + AB - 1) / AB), dim3(128), smem, a,
+                          (const uint8_t *)a.ukv->rec, a.ukv->kc, rows));
     QB_LAUNCHED(ctx, "latent_absorb_kernel");
-    // one span over everything when the rows alone fill the GPU, fixed spans otherwise
-    const bool one = a.R > QB_LAT_ABSORB_ROWS;
-    const uint32_t span = one ? (a.max_pos + 63) / 64 * 64 : QB_LAT_SPLIT, n_splits = one ? 1 : (a.max_pos + QB_LAT_SPLIT - 1) / QB_LAT_SPLIT;
-    const uint32_t MT = a.R * a.H > 16 ? 2 : 1;
-    if (!a.f32 && a.rankp() <= 512 && split_smem(a.pitch(), MT).total <= 227 * 1024) {
-        if (MT == 2) QB_TRY(launch_split_nv<2>(ctx, a, span, n_splits));
-        else QB_TRY(launch_split_nv<1>(ctx, a, span, n_splits));
-    } else {
-        QB_TRY(launch_simt<T>(ctx, a, span, n_splits));
-    }
-    const size_t sm_m = (((size_t)n_splits + 3) / 4 * 4 + kc * 64) * sizeof(float);
-    QB_REQUIRE(sm_m <= 227 * 1024, "latent attention: %u spans do not fit", n_splits);
-    QB_CUDA(cudaFuncSetAttribute(latent_merge_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sm_m));
-    const uint32_t vz = std::max(1u, std::min((a.vdim + 7) / 8, (2u * (uint32_t)ctx->sm_count) / std::max(1u, a.H * rows)));
-    QB_CUDA(qb_launch_pdl(ctx->stream, latent_merge_kernel<T>, dim3(a.H, rows, vz), dim3(LT), sm_m, a, (const uint8_t *)a.ukv->rec, kc, span, n_splits));
+    return QB_OK;
+}
+template <typename T, int MB>
+int launch_merge(qb_ctx *ctx, const QbLatent &a, uint32_t rows, uint32_t n_splits) {
+    const uint32_t kc = a.ukv->kc, groups = (rows + MB - 1) / MB;
+    const size_t smem = (((size_t)MB * n_splits + 3) / 4 * 4 + MB * kc * 64) * sizeof(float);
+    QB_REQUIRE(smem <= 227 * 1024, "latent attention: a latent of %u does not fit", a.rank);
+    QB_CUDA(cudaFuncSetAttribute(latent_merge_kernel<T, MB>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    const uint32_t vz = std::max(1u, std::min((a.vdim + 31) / 32, (4u * (uint32_t)ctx->sm_count + a.H * groups - 1) / (a.H * groups)));
+    QB_CUDA(qb_launch_pdl(ctx->stream, latent_merge_kernel<T, MB>, dim3(a.H, groups, vz), dim3(LT), smem, a, (const uint8_t *)a.ukv->rec, kc, rows, n_splits));
     QB_LAUNCHED(ctx, "latent_merge_kernel");
     return QB_OK;
 }
 
+template <typename T>
+int latent_absorbed(qb_ctx *ctx, QbLatent a) {
+    const uint32_t rows = a.ns * a.R;
+    if (a.R > QB_LAT_ABSORB_ROWS) a.max_splits = 1;          // the rows alone fill the GPU
+    const uint32_t n_splits = std::min(a.max_splits, (a.max_pos + 63) / 64);
+    if (rows == 1) QB_TRY((launch_absorb<T, 1>(ctx, a, rows)));
+    else QB_TRY((launch_absorb<T, 8>(ctx, a, rows)));
+    const uint32_t MT = a.R * a.H > 16 ? 2 : 1;
+    static const bool use_tc = qb_env_u32("QW3B200_LATENT_TC", 1) != 0;       // 0: the mma.sync form, for comparison
+    if (use_tc && a.R <= QB_LAT_ABSORB_ROWS && qb_latent_tc_supports(a)) {
+        QB_TRY(qb_launch_latent_split_tc(ctx, a, n_splits));
+    } else if (!a.f32 && a.rankp() <= 512 && split_smem(a.pitch(), MT).total <= 227 * 1024) {
+        if (MT == 2) QB_TRY(launch_split_nv<2>(ctx, a, n_splits));
+        else QB_TRY(launch_split_nv<1>(ctx, a, n_splits));
+    } else {
+        QB_TRY(launch_simt<T>(ctx, a, n_splits));
+    }
+    if (rows == 1) return launch_merge<T, 1>(ctx, a, rows, n_splits);
+    return launch_merge<T, 4>(ctx, a, rows, n_splits);
+}
+
 }  // namespace
+
+uint32_t qb_latent_max_splits(const QbLatent &a, uint32_t ns, uint32_t sms) {
+    const uint32_t groups = (a.H + 47) / 48;
+    return std::max(1u, std::min(64u, sms / (ns * groups)));
+}
 
 bool qb_latent_expands(const QbLatent &a) {
     return !a.f32 && a.vdimp() <= 256 && ((size_t)(128 + 128) * (a.dimp() + a.rotp() + 8) + 128 * (a.vdimp() + 8)) * 2 <= 227 * 1024;
 }
 
-size_t qb_latent_part_floats(const QbLatent &a, uint32_t rows_cap, uint32_t n_seqs, uint32_t max_keys) {
-    const size_t splits = (max_keys + QB_LAT_SPLIT - 1) / QB_LAT_SPLIT;
-    const size_t few = (size_t)std::max(n_seqs, QB_LAT_ABSORB_ROWS) * splits;
+size_t qb_latent_part_floats(const QbLatent &a, uint32_t rows_cap, uint32_t n_seqs, uint32_t sms) {
+    const size_t few = std::max({n_seqs, sms, QB_LAT_ABSORB_ROWS * 64u});       // (sequences x rows each) x spans
     return std::max(few, qb_latent_expands(a) ? (size_t)0 : (size_t)rows_cap) * a.H * a.rank;
 }
 
-int qb_launch_latent(qb_ctx *ctx, const QbLatent &a) {
+int qb_launch_latent(qb_ctx *ctx, const QbLatent &args) {
+    QbLatent a = args;
+    a.err_flag = ctx->err_flag_dev;
     const uint32_t rows = a.ns * a.R;
     QB_REQUIRE(rows > 0 && a.rot.dims <= a.rot_dim && a.rot.dims % 2 == 0 && a.stride == a.H * (a.dim + a.rot_dim) + a.rank + a.rot_dim, "latent attention: bad arguments");
     const size_t sm_p = ((size_t)a.rot.dims + a.rank) * sizeof(float);
-    if (a.f32) QB_CUDA(qb_launch_pdl(ctx->stream, latent_prepare_kernel<float>, dim3(rows), dim3(LT), sm_p, a, ctx->err_flag_dev));
-    else QB_CUDA(qb_launch_pdl(ctx->stream, latent_prepare_kernel<__nv_bfloat16>, dim3(rows), dim3(LT), sm_p, a, ctx->err_flag_dev));
+    // query heads per CTA: enough elements for its threads, fewer when there are few rows
+    const uint32_t per = a.dimp() + a.rotp(), hpb = std::max(1u, (rows <= 64 ? 1024u : 4096u) / per);
+    const dim3 grid(rows, 1 + (a.H + hpb - 1) / hpb);
+    if (a.f32) QB_CUDA(qb_launch_pdl(ctx->stream, latent_prepare_kernel<float>, grid, dim3(LT), sm_p, a, hpb));
+    else QB_CUDA(qb_launch_pdl(ctx->stream, latent_prepare_kernel<__nv_bfloat16>, grid, dim3(LT), sm_p, a, hpb));
     QB_LAUNCHED(ctx, "latent_prepare_kernel");
     if (a.f32) return latent_absorbed<float>(ctx, a);
     if (!a.ingest || a.R <= QB_LAT_ABSORB_ROWS || !qb_latent_expands(a)) return latent_absorbed<__nv_bfloat16>(ctx, a);

@@ -31,6 +31,17 @@ __device__ __forceinline__ void qb_rot_pair(const QbRotary &r, uint32_t j, uint3
     if (r.interleaved) { i = j >> 1; partner = j ^ 1; first = !(j & 1); }
     else { const uint32_t h = r.dims / 2; first = j < h; i = first ? j : j - h; partner = first ? j + h : j - h; }
 }
+// Sum of up to 8 K-segment partials of one product, ascending, with every load in flight.
+__device__ __forceinline__ float qb_sum8(const float *p, size_t idx, uint32_t S, size_t pstride) {
+    if (S == 1) return p[idx];
+    float v[8];
+#pragma unroll
+    for (uint32_t s = 0; s < 8; ++s) v[s] = s < S ? p[idx + s * pstride] : 0.0f;
+    float t = v[0];
+#pragma unroll
+    for (uint32_t s = 1; s < 8; ++s) t += v[s];
+    return t;
+}
 // Sum over a block of `nwarps` warps; every thread returns it.  red: nwarps floats of shared memory.
 __device__ __forceinline__ float qb_block_sum(float v, float *red, uint32_t nwarps) {
     v = warp_sum(v);
@@ -98,6 +109,7 @@ struct QbLatent {
     uint32_t pt_stride = 0, page_size = 0, max_pos = 0;
     void *cache = nullptr;                    // [slot][rankp + rotp], activation type
     bool ingest = false;                      // a prompt chunk of one sequence
+    uint32_t max_splits = 1;                  // spans a sequence's keys are cut into at most (absorbed form)
     // scratch (sizes: QbLatentScratch)
     void *q = nullptr, *qa = nullptr;
     float *part_acc = nullptr, *part_ml = nullptr;
@@ -105,6 +117,7 @@ struct QbLatent {
     __nv_bfloat16 *kr = nullptr, *kv = nullptr;
     QbActBuf out;                             // [rows][H*vdim]
     bool f32 = false;
+    int *err_flag = nullptr;
     __host__ __device__ uint32_t dimp() const { return (dim + 15) & ~15u; }
     __host__ __device__ uint32_t rotp() const { return (rot_dim + 15) & ~15u; }
     __host__ __device__ uint32_t vdimp() const { return (vdim + 15) & ~15u; }
@@ -112,9 +125,18 @@ struct QbLatent {
     __host__ __device__ uint32_t pitch() const { return rankp() + rotp(); }
 };
 static const uint32_t QB_LAT_ABSORB_ROWS = 16;     // rows per sequence up to which the absorbed form runs
-static const uint32_t QB_LAT_SPLIT = 128;          // keys per split of the absorbed form
+#ifdef __CUDACC__
+// Keys per span of a sequence's absorbed attention: its keys over at most max_splits spans of whole 64-key tiles.  A function
+// of the sequence's own length and of how many sequences share the launch; where the cuts fall changes rounding only.
+__device__ __forceinline__ uint32_t qb_latent_span(uint32_t keys, uint32_t max_splits) { return ((keys + max_splits - 1) / max_splits + 63) & ~63u; }
+#endif
 // Whether prompt chunks of this shape expand keys and values (bfloat16, sizes within the kernel's registers).
 bool qb_latent_expands(const QbLatent &a);
-// Floats of part_acc for up to `rows_cap` prompt rows / n_seqs decode rows with max_keys keys.
-size_t qb_latent_part_floats(const QbLatent &a, uint32_t rows_cap, uint32_t n_seqs, uint32_t max_keys);
+// The absorbed form's spans on tcgen05 (latent_attention_tc.cu): bfloat16, 16-key pages, a latent of at most 512.
+bool qb_latent_tc_supports(const QbLatent &a);
+int qb_launch_latent_split_tc(qb_ctx *ctx, const QbLatent &a, uint32_t n_splits);
+// Spans per sequence that fill the GPU once with ns sequences in the launch.
+uint32_t qb_latent_max_splits(const QbLatent &a, uint32_t ns, uint32_t sms);
+// Floats of part_acc for up to rows_cap prompt rows / n_seqs decode rows.
+size_t qb_latent_part_floats(const QbLatent &a, uint32_t rows_cap, uint32_t n_seqs, uint32_t sms);
 int qb_launch_latent(qb_ctx *ctx, const QbLatent &a);

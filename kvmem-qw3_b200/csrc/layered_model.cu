@@ -382,7 +382,7 @@ int layered_batch_alloc(qb_ctx *ctx, qb_batch *b, size_t slots) {
         const QbLatent a = latent_shape(S.mixer, f32);
         q = std::max(q, (size_t)rows * a.H * (a.dimp() + a.rotp()));
         qa = std::max(qa, (size_t)rows * a.H * a.pitch());
-        const size_t pf = qb_latent_part_floats(a, rows, b->n_seqs, max_keys);
+        const size_t pf = qb_latent_part_floats(a, rows, b->n_seqs, sms);
         acc = std::max(acc, pf);
         ml = std::max(ml, pf / a.rank * 2);
         if (qb_latent_expands(a)) {
@@ -391,9 +391,9 @@ int layered_batch_alloc(qb_ctx *ctx, qb_batch *b, size_t slots) {
             kv = std::max(kv, (size_t)max_keys * L.w_ukv.rows);
         }
     }
-    QB_TRY(qb_act_alloc(&B->x, rows, D, f32));
-    QB_TRY(qb_act_alloc(&B->mix, rows, mix, f32));
-    QB_TRY(qb_act_alloc(&B->ff, rows, ff, f32));
+    QB_TRY(qb_act_alloc(ctx, &B->x, rows, D, f32));
+    QB_TRY(qb_act_alloc(ctx, &B->mix, rows, mix, f32));
+    QB_TRY(qb_act_alloc(ctx, &B->ff, rows, ff, f32));
     QB_CUDA(cudaMalloc(&B->parts, parts * sizeof(float)));
     QB_CUDA(cudaMalloc(&B->emb, (size_t)rows * D * sizeof(float)));
     if (q) {
@@ -403,7 +403,7 @@ int layered_batch_alloc(qb_ctx *ctx, qb_batch *b, size_t slots) {
         QB_CUDA(cudaMalloc(&B->part_ml, ml * sizeof(float)));
     }
     if (kv) {
-        QB_TRY(qb_act_alloc(&B->lat, max_keys, (uint32_t)lat_ld, false));
+        QB_TRY(qb_act_alloc(ctx, &B->lat, max_keys, (uint32_t)lat_ld, false));
         QB_CUDA(cudaMalloc(&B->kr, kr * 2));
         QB_CUDA(cudaMalloc(&B->kv, kv * 2));
     }
@@ -474,6 +474,7 @@ int latent_block(qb_ctx *ctx, qb_batch *b, uint32_t run, const RowSet &rs, uint3
     a.seq_pos = rs.seq_pos; a.max_pos = rs.max_pos; a.ingest = rs.ingest;
     a.page_table = b->page_table + (size_t)rs.seq0 * b->pages_per_seq; a.pt_stride = b->pages_per_seq; a.page_size = b->page_size;
     a.cache = B->cache[run];
+    a.max_splits = qb_latent_max_splits(a, rs.ns, (uint32_t)ctx->sm_count);
     a.q = B->q; a.qa = B->qa; a.part_acc = B->part_acc; a.part_ml = B->part_ml; a.lat = B->lat; a.kr = B->kr; a.kv = B->kv;
     a.out = B->mix;
     QB_TRY(qb_launch_latent(ctx, a));

@@ -100,6 +100,7 @@ struct qb_ctx {
 int qb_ctx_scratch(qb_ctx *ctx, size_t bytes, void **out);
 int qb_ctx_scratch2(qb_ctx *ctx, size_t bytes, void **out);
 void qb_trace_mark(qb_ctx *ctx, const char *name);
+uint32_t qb_env_u32(const char *name, uint32_t dflt);
 // Device timeline (qb_debug_timeline_*): while enabled every tensor-core GEMM launch gets a slot of
 // QB_TL_CTAS x 4 words; CTA b stores {entry, dependency wait passed, exit} in nanoseconds of the global
 // timer and its SM id.  Returns null when disabled or full.

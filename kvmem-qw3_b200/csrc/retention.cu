@@ -17,9 +17,15 @@ namespace {
 constexpr int RT = 256;
 constexpr uint32_t C = QB_RET_CHUNK, VCH = 32;
 
+// "This CTA runs": arrived at on entry, awaited before the first store into another CTA's shared memory, which must not be
+// touched before that CTA has started.
+__device__ __forceinline__ void cluster_started() { asm volatile("barrier.cluster.arrive.relaxed.aligned;" ::: "memory"); }
+__device__ __forceinline__ void cluster_wait_started() { asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory"); }
+
 template <typename T>
 __global__ void __launch_bounds__(RT)
 retention_step_kernel(QbRetention a, uint32_t vc) {
+    cluster_started();
     QB_PDL_ENTER();
     cg::cluster_group cl = cg::this_cluster();
     extern __shared__ float sm[];
@@ -46,11 +52,11 @@ retention_step_kernel(QbRetention a, uint32_t vc) {
         for (uint32_t i = tid; i < half; i += RT) qb_rot_angle(a.rot, pos, i, cs[i], sn[i]);
         __syncthreads();
         for (uint32_t d = tid; d < a.dim; d += RT) {
-            float q = qb_ldsum(a.proj, base + h * a.dim + d, a.S, ps), k = qb_ldsum(a.proj, base + kb + h * a.dim + d, a.S, ps);
+            float q = qb_sum8(a.proj, base + h * a.dim + d, a.S, ps), k = qb_sum8(a.proj, base + kb + h * a.dim + d, a.S, ps);
             if (d < a.rot.dims) {
                 uint32_t i, p; bool first;
                 qb_rot_pair(a.rot, d, i, p, first);
-                const float q2 = qb_ldsum(a.proj, base + h * a.dim + p, a.S, ps), k2 = qb_ldsum(a.proj, base + kb + h * a.dim + p, a.S, ps);
+                const float q2 = qb_sum8(a.proj, base + h * a.dim + p, a.S, ps), k2 = qb_sum8(a.proj, base + kb + h * a.dim + p, a.S, ps);
                 q = first ? q * cs[i] - q2 * sn[i] : q * cs[i] + q2 * sn[i];
                 k = first ? k * cs[i] - k2 * sn[i] : k * cs[i] + k2 * sn[i];
             }
@@ -60,7 +66,7 @@ retention_step_kernel(QbRetention a, uint32_t vc) {
         __syncthreads();
         const uint32_t rg = tid >> 5;
         for (uint32_t c = tid & 31; c < vc; c += 32) {
-            const float v = c < nv ? qb_ldsum(a.proj, base + vb + h * a.vdim + v0 + c, a.S, ps) : 0.0f;
+            const float v = c < nv ? qb_sum8(a.proj, base + vb + h * a.vdim + v0 + c, a.S, ps) : 0.0f;
             float o = 0.0f;
 #pragma unroll 4
             for (uint32_t d = rg; d < a.dim; d += RT / 32) {
@@ -71,6 +77,7 @@ retention_step_kernel(QbRetention a, uint32_t vc) {
             red[rg * vc + c] = o;
         }
         __syncthreads();
+        if (r == 0) cluster_wait_started();
         if (tid < 32) {
             float ss = 0.0f;
             for (uint32_t c = tid; c < vc; c += 32) {
@@ -89,7 +96,7 @@ retention_step_kernel(QbRetention a, uint32_t vc) {
         const float inv = rsqrtf(tot / (float)a.vdim + a.eps);
         T *out = (T *)a.out.p + m * a.out.ld + h * a.vdim + v0;
         for (uint32_t c = tid; c < nv; c += RT) {
-            const float g = qb_ldsum(a.proj, base + gb + h * a.vdim + v0 + c, a.S, ps);
+            const float g = qb_sum8(a.proj, base + gb + h * a.vdim + v0 + c, a.S, ps);
             out[c] = qb_cast<T>(red[c] * inv * qb_swiglu(g, 1.0f));
         }
         __syncthreads();
@@ -99,6 +106,103 @@ retention_step_kernel(QbRetention a, uint32_t vc) {
         if (c < nv) gst[(size_t)d * a.vdim + c] = st[i];
     }
     cl.sync();                                       // no CTA leaves while a peer may still write its xch
+}
+
+// One row per sequence (plain decode): the state never leaves the registers -- a thread holds NI pieces of four value
+// columns, all requested at once before the row's q and k are rotated.  Needs vdim and the projection offsets to be
+// multiples of 4.
+template <typename T, int NI>
+__global__ void __launch_bounds__(RT)
+retention_decode_kernel(QbRetention a, uint32_t vc) {
+    cluster_started();
+    QB_PDL_ENTER();
+    cg::cluster_group cl = cg::this_cluster();
+    extern __shared__ float sm[];
+    float *qs = sm, *ks = qs + a.dim;
+    float4 *red = reinterpret_cast<float4 *>(ks + a.dim);      // [RT / 32 warps][vc / 4]   (dim is even: 16-byte aligned)
+    __shared__ float xch[16], part[RT / 32];
+    const uint32_t tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, h = blockIdx.y, m = blockIdx.z, v0 = blockIdx.x * vc;
+    const uint32_t nv = min(vc, a.vdim - v0), g4 = vc / 4, c4 = tid % g4, dg = tid / g4, nd = RT / g4;
+    const size_t base = (size_t)m * a.stride, ps = (size_t)a.ns * a.stride;
+    const bool on = c4 * 4 < nv;
+    float *gst = a.state + ((size_t)m * a.H + h) * a.dim * a.vdim + v0 + c4 * 4;
+    float4 st[NI];
+#pragma unroll
+    for (int i = 0; i < NI; ++i) {
+        const uint32_t d = dg + i * nd;
+        st[i] = on && d < a.dim ? *reinterpret_cast<const float4 *>(gst + (size_t)d * a.vdim) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+    const uint32_t kb = a.H * a.dim, vb = 2 * kb, gb = vb + a.H * a.vdim;
+    const float decay = a.powers[h * (C + 1) + 1], kscale = 1.0f / sqrtf((float)a.dim);
+    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (on) {
+        const float *p = a.proj + base + vb + h * a.vdim + v0 + c4 * 4;
+        v = *reinterpret_cast<const float4 *>(p);
+        for (uint32_t s = 1; s < a.S; ++s) {
+            const float4 w = *reinterpret_cast<const float4 *>(p + s * ps);
+            v.x += w.x; v.y += w.y; v.z += w.z; v.w += w.w;
+        }
+    }
+    const int pos = a.seq_pos[m];
+    for (uint32_t t = tid; t < 2 * a.dim; t += RT) {           // q, then k: a pair's two threads each take one element
+        const bool is_k = t >= a.dim;
+        const uint32_t d = is_k ? t - a.dim : t;
+        const size_t at = base + (is_k ? kb : 0) + h * a.dim;
+        float u = qb_sum8(a.proj, at + d, a.S, ps);
+        if (d < a.rot.dims) {
+            uint32_t i, p; bool first;
+            qb_rot_pair(a.rot, d, i, p, first);
+            const float w = qb_sum8(a.proj, at + p, a.S, ps);
+            float c, sn;
+            qb_rot_angle(a.rot, pos, i, c, sn);
+            u = first ? u * c - w * sn : u * c + w * sn;
+        }
+        sm[t] = is_k ? u * kscale : u;
+    }
+    __syncthreads();
+    float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+    for (int i = 0; i < NI; ++i) {
+        const uint32_t d = dg + i * nd;
+        if (d < a.dim) {
+            const float q = qs[d], k = ks[d];
+            st[i].x = fmaf(st[i].x, decay, k * v.x); st[i].y = fmaf(st[i].y, decay, k * v.y);
+            st[i].z = fmaf(st[i].z, decay, k * v.z); st[i].w = fmaf(st[i].w, decay, k * v.w);
+            if (on) *reinterpret_cast<float4 *>(gst + (size_t)d * a.vdim) = st[i];
+            o.x = fmaf(st[i].x, q, o.x); o.y = fmaf(st[i].y, q, o.y); o.z = fmaf(st[i].z, q, o.z); o.w = fmaf(st[i].w, q, o.w);
+        }
+    }
+    for (uint32_t off = g4; off < 32; off <<= 1) {             // lanes of a warp that hold the same columns
+        o.x += __shfl_xor_sync(0xffffffffu, o.x, off); o.y += __shfl_xor_sync(0xffffffffu, o.y, off);
+        o.z += __shfl_xor_sync(0xffffffffu, o.z, off); o.w += __shfl_xor_sync(0xffffffffu, o.w, off);
+    }
+    if (lane < g4) red[warp * g4 + lane] = o;
+    __syncthreads();
+    float out = 0.0f;
+    if (tid < vc) {
+        const float *r = reinterpret_cast<const float *>(red);
+#pragma unroll
+        for (uint32_t w = 0; w < RT / 32; ++w) out += r[w * vc + tid];
+    }
+    const float ss = warp_sum(out * out);                       // columns past vdim are zero
+    if (lane == 0) part[warp] = ss;
+    __syncthreads();
+    const uint32_t csize = cl.num_blocks();
+    float tot = 0.0f;
+#pragma unroll
+    for (uint32_t w = 0; w < RT / 32; ++w) tot += part[w];
+    cluster_wait_started();
+    if (csize > 1) {
+        if (tid < csize) cl.map_shared_rank(xch, tid)[cl.block_rank()] = tot;
+        cl.sync();
+        tot = 0.0f;
+        for (uint32_t i = 0; i < csize; ++i) tot += xch[i];
+    }
+    const float inv = rsqrtf(tot / (float)a.vdim + a.eps);
+    if (tid < nv) {
+        const float g = qb_sum8(a.proj, base + gb + h * a.vdim + v0 + tid, a.S, ps);
+        ((T *)a.out.p + (size_t)m * a.out.ld + h * a.vdim + v0)[tid] = qb_cast<T>(out * inv * qb_swiglu(g, 1.0f));
+    }
 }
 
 // Rotates q and k of a prompt chunk in place (k also scaled); adds K-segment partial sums of every column first.
@@ -118,7 +222,7 @@ retention_rotate_kernel(QbRetention a) {
     for (uint32_t t = threadIdx.x; t < 2 * a.H * half; t += RT) {
         const uint32_t i = t % half, hh = t / half;                           // hh < H: q heads, then k heads
         const uint32_t j = hh * a.dim + (a.rot.interleaved ? 2 * i : i), p = a.rot.interleaved ? j + 1 : j + half;
-        const float u = qb_ldsum(a.proj, base + j, a.S, ps), v = qb_ldsum(a.proj, base + p, a.S, ps), sc = hh < a.H ? 1.0f : kscale;
+        const float u = qb_sum8(a.proj, base + j, a.S, ps), v = qb_sum8(a.proj, base + p, a.S, ps), sc = hh < a.H ? 1.0f : kscale;
         row[j] = (u * cs[i] - v * sn[i]) * sc;
         row[p] = (v * cs[i] + u * sn[i]) * sc;
     }
@@ -126,10 +230,10 @@ retention_rotate_kernel(QbRetention a) {
     const uint32_t rest = a.dim - a.rot.dims;
     for (uint32_t t = threadIdx.x; t < 2 * a.H * rest; t += RT) {
         const uint32_t hh = t / rest, j = hh * a.dim + a.rot.dims + t % rest;
-        row[j] = qb_ldsum(a.proj, base + j, a.S, ps) * (hh < a.H ? 1.0f : kscale);
+        row[j] = qb_sum8(a.proj, base + j, a.S, ps) * (hh < a.H ? 1.0f : kscale);
     }
     if (a.S > 1)
-        for (uint32_t j = 2 * a.H * a.dim + threadIdx.x; j < a.stride; j += RT) row[j] = qb_ldsum(a.proj, base + j, a.S, ps);
+        for (uint32_t j = 2 * a.H * a.dim + threadIdx.x; j < a.stride; j += RT) row[j] = qb_sum8(a.proj, base + j, a.S, ps);
 }
 
 // grid (value slices, H, sequences).  q and k are rotated and scaled; the outputs replace the v columns of the projection.
@@ -281,14 +385,11 @@ retention_gate_kernel(QbRetention a) {
     for (uint32_t c = lane; c < a.vdim; c += 32) out[c] = qb_cast<T>(o[c] * inv * qb_swiglu(g[c], 1.0f));
 }
 
-template <typename T>
-int launch_step(qb_ctx *ctx, const QbRetention &a) {
-    uint32_t vc = VCH;
-    while ((a.vdim + vc - 1) / vc > 8) vc += VCH;
+template <typename K>
+int launch_cluster(qb_ctx *ctx, K kernel, const QbRetention &a, uint32_t vc, size_t smem, const char *name) {
     const uint32_t split = (a.vdim + vc - 1) / vc;
-    const size_t smem = ((size_t)a.dim * vc + 2 * a.dim + a.rot.dims + (RT / 32) * vc) * sizeof(float);
     QB_REQUIRE(smem <= 220 * 1024, "retention: head of %u x %u does not fit", a.dim, a.vdim);
-    QB_CUDA(cudaFuncSetAttribute(retention_step_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    QB_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
     cudaLaunchConfig_t cfg = {};
     cfg.gridDim = dim3(split, a.H, a.ns);
     cfg.blockDim = dim3(RT);
@@ -301,9 +402,28 @@ int launch_step(qb_ctx *ctx, const QbRetention &a) {
     attr[1].val.programmaticStreamSerializationAllowed = 1;
     cfg.attrs = attr;
     cfg.numAttrs = 2;
-    QB_CUDA(cudaLaunchKernelEx(&cfg, retention_step_kernel<T>, a, vc));
-    QB_LAUNCHED(ctx, "retention_step_kernel");
+    QB_CUDA(cudaLaunchKernelEx(&cfg, kernel, a, vc));
+    QB_LAUNCHED(ctx, name);
     return QB_OK;
+}
+
+template <typename T>
+int launch_step(qb_ctx *ctx, const QbRetention &a) {
+    if (a.R == 1 && a.vdim % 4 == 0 && a.dim % 2 == 0 && (a.H * a.dim) % 2 == 0) {
+        // slices of 32 columns spread a few heads over the SMs; with many (sequence, head) pairs a CTA takes 128
+        const uint32_t vc = (uint64_t)a.ns * a.H >= 2u * (uint32_t)ctx->sm_count && a.vdim > 32 ? 128 : 32;
+        const uint32_t ni = (a.dim + RT / (vc / 4) - 1) / (RT / (vc / 4)), split = (a.vdim + vc - 1) / vc;
+        const size_t smem = ((size_t)2 * a.dim + (RT / 32) * vc) * sizeof(float);
+        if (split <= 8 && ni <= 16) {
+            if (ni <= 2) return launch_cluster(ctx, retention_decode_kernel<T, 2>, a, vc, smem, "retention_decode_kernel");
+            if (ni <= 4) return launch_cluster(ctx, retention_decode_kernel<T, 4>, a, vc, smem, "retention_decode_kernel");
+            if (ni <= 8) return launch_cluster(ctx, retention_decode_kernel<T, 8>, a, vc, smem, "retention_decode_kernel");
+            return launch_cluster(ctx, retention_decode_kernel<T, 16>, a, vc, smem, "retention_decode_kernel");
+        }
+    }
+    uint32_t vc = VCH;
+    while ((a.vdim + vc - 1) / vc > 8) vc += VCH;
+    return launch_cluster(ctx, retention_step_kernel<T>, a, vc, ((size_t)a.dim * vc + 2 * a.dim + a.rot.dims + (RT / 32) * vc) * sizeof(float), "retention_step_kernel");
 }
 
 }  // namespace

@@ -169,6 +169,22 @@ def test_sizes_beyond_the_tiled_kernels(make, layer, dtype):
     b.close()
 
 
+@pytest.mark.parametrize("heads,rank,rot_dim,n_seqs", [(20, 512, 64, 40), (50, 128, 16, 1), (1, 256, 32, 40), (7, 96, 16, 3), (34, 448, 80, 40)])
+def test_absorbed_attention_shapes(make, heads, rank, rot_dim, n_seqs):
+    """Decode rows over many keys, at several head counts and latent sizes; a large batch cuts a sequence into few spans of
+    several 128-key tiles, and a raised scale lets the running maximum grow from tile to tile."""
+    c = make(config([lat(heads=heads, dim=16, rot_dim=rot_dim, rot=rot_dim, vdim=24, rank=rank, scale=0.7, ff=None)]))
+    n = 1300 if n_seqs == 40 else 333
+    toks = c.tokens(n + 6)
+    want = c.want(toks)[n:]
+    b = c.batch("bfloat16", n_seqs=n_seqs, max_ctx=1400, pool_pages=100)
+    b.prefill(n_seqs - 1, toks[:n], more=True)
+    got = [b.score(n_seqs - 1, [t], [0]) for t in toks[n:n + 3]]
+    got.append(b.score(n_seqs - 1, toks[n + 3:], range(3)))
+    close_to(np.concatenate(got), want, "bfloat16")
+    b.close()
+
+
 # ---- schedules ---------------------------------------------------------------------------------------------------------------
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
 @pytest.mark.parametrize("size", [1, 2, 3, 15, 16, 17, 63, 64, 65, 129, [2, 100, 3, 1, 17]])
