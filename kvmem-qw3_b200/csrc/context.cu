@@ -33,6 +33,7 @@ extern "C" int qb_create(int device, qb_ctx **out) {
     qb_ctx *ctx = new qb_ctx();
     ctx->device = device;
     ctx->sm_count = prop.multiProcessorCount;
+    ctx->sync_launches = qb_env_u32("QW3B200_SYNC_LAUNCHES", 0) != 0;
     QB_CUDA(cudaStreamCreateWithFlags(&ctx->stream, cudaStreamNonBlocking));
     std::vector<float> table(QS_NORMAL_TABLE_SIZE);
     qs_build_normal_table(table.data());
@@ -63,7 +64,7 @@ extern "C" int qb_synchronize(qb_ctx *ctx) {
     QB_CUDA(cudaMemcpy(&flag, ctx->err_flag_dev, sizeof(int), cudaMemcpyDeviceToHost));
     if (flag != 0) {
         cudaMemset(ctx->err_flag_dev, 0, sizeof(int));
-        return qb_fail(QB_ERR_CUDA, "a kernel recorded an error (code %d: 3001 / 3002 = a K/V append to an unassigned page, skipped; other codes = a bounded wait that ran out)", flag);
+        return qb_fail(QB_ERR_CUDA, "a kernel recorded an error (code %d: 3001 / 3002 = a K/V append to an unassigned page, skipped; 6001 = a row outside the batch; other codes = a bounded wait that ran out)", flag);
     }
     return QB_OK;
 }

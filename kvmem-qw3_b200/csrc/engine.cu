@@ -464,7 +464,7 @@ static int batch_create(qb_ctx *ctx, qb_model *m, uint32_t n_seqs, uint32_t max_
     b->logit_rows = n_seqs * (draft_k + 1);
     b->rows_cap = std::max(b->chunk, b->logit_rows);
     const uint32_t H = c.n_embd, K1 = draft_k + 1, rows = b->rows_cap;
-    const size_t slots = (size_t)(pool_pages ? pool_pages : n_seqs * b->pages_per_seq) * page_size;
+    const size_t slots = b->slots = (size_t)(pool_pages ? pool_pages : n_seqs * b->pages_per_seq) * page_size;
     // page table: identity / reverse / seeded shuffle over the whole pool
     {
         const size_t total = (size_t)n_seqs * b->pages_per_seq;

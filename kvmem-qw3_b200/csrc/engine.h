@@ -88,6 +88,7 @@ struct qb_batch {
     qb_model *m = nullptr;
     QbLayeredBatch *layered = nullptr;     // a layered model's caches and activations (layered_model.cu)
     std::vector<StateBlock> blocks;        // recurrent state of every kind: reset, swap, snapshot and prefix entries walk this list
+    size_t slots = 0;                      // K/V positions the paged caches hold
     uint32_t n_seqs = 0, max_ctx = 0, k = 0, page_size = 0, pages_per_seq = 0, rows_cap = 0, chunk = 0, logit_rows = 0;
     bool attn_tc = false;                  // decode / verify attention on the tensor-memory kernel: decided once, from n_seqs * max_ctx
     uint32_t attn_split = 0;               // keys per attention split of this batch (absolute boundaries): decided once with attn_tc

@@ -63,12 +63,12 @@ latent_prepare_kernel(QbLatent a, uint32_t hpb) {
         ss += v * v;
     }
     const float inv = rsqrtf(qb_block_sum(ss, red, LT / 32) / (float)a.rank + a.eps);
-    const int32_t page = a.page_table[(size_t)s * a.pt_stride + (uint32_t)pos / a.page_size];
-    if (page < 0) {
+    const int64_t at = qb_latent_slot(a, a.page_table + (size_t)s * a.pt_stride, (uint32_t)pos);
+    if (at < 0) {
         if (tid == 0) atomicExch(a.err_flag, 3002);                    // an unassigned page: nothing is appended
         return;
     }
-    T *slot = (T *)a.cache + ((size_t)page * a.page_size + (uint32_t)pos % a.page_size) * a.pitch();
+    T *slot = (T *)a.cache + (size_t)at * a.pitch();
     const uint32_t rp = a.rankp();
     for (uint32_t i = tid; i < a.pitch(); i += LT) {
         float v = 0.0f;
@@ -162,7 +162,8 @@ latent_split_simt_kernel(QbLatent a, uint32_t n_splits) {
             const uint32_t j = i / D, e = i % D;
             const int key = kt + (int)j;
             float v = 0.0f;
-            if (key < k_end) v = qb_f32(((const T *)a.cache)[((size_t)pt[(uint32_t)key / a.page_size] * a.page_size + (uint32_t)key % a.page_size) * D + e]);
+            const int64_t at = key < k_end ? qb_latent_slot(a, pt, (uint32_t)key) : -1;
+            if (at >= 0) v = qb_f32(((const T *)a.cache)[(size_t)at * D + e]);
             ts[j * DP + e] = v;
         }
         __syncthreads();
@@ -272,10 +273,8 @@ latent_split_kernel(QbLatent a, uint32_t n_splits) {
         for (uint32_t i = tid; i < DKT * (D / 8); i += LT) {
             const uint32_t j = i / (D / 8), c = i % (D / 8);
             const int key = kt + (int)j;
-            const bool ok = key < k_end;
-            const __nv_bfloat16 *src = cache;
-            if (ok) src += ((size_t)pt[(uint32_t)key / a.page_size] * a.page_size + (uint32_t)key % a.page_size) * D + c * 8;
-            cp16(dst + j * pitch + c * 16, src, ok);
+            const int64_t at = key < k_end ? qb_latent_slot(a, pt, (uint32_t)key) : -1;
+            cp16(dst + j * pitch + c * 16, at >= 0 ? cache + (size_t)at * D + c * 8 : cache, at >= 0);
         }
         cp_commit();
     };
@@ -479,8 +478,8 @@ latent_gather_kernel(QbLatent a, uint32_t n) {
     const uint64_t i = (uint64_t)blockIdx.x * LT + threadIdx.x;
     if (i >= (uint64_t)n * D8) return;
     const uint32_t key = (uint32_t)(i / D8), c = (uint32_t)(i % D8);
-    const uint4 v = *reinterpret_cast<const uint4 *>((const __nv_bfloat16 *)a.cache +
-                                                     ((size_t)a.page_table[key / a.page_size] * a.page_size + key % a.page_size) * a.pitch() + c * 8);
+    const int64_t at = qb_latent_slot(a, a.page_table, key);
+    const uint4 v = at >= 0 ? *reinterpret_cast<const uint4 *>((const __nv_bfloat16 *)a.cache + (size_t)at * a.pitch() + c * 8) : make_uint4(0u, 0u, 0u, 0u);
     if (c < r8) *reinterpret_cast<uint4 *>((__nv_bfloat16 *)a.lat.p + (size_t)key * a.lat.ld + c * 8) = v;
     else *reinterpret_cast<uint4 *>(a.kr + (size_t)key * a.rotp() + (c - r8) * 8) = v;
 }

@@ -95,7 +95,7 @@ latent_split_tc_kernel(QbLatent a, const __grid_constant__ CUtensorMap map, uint
         const int32_t *pt = a.page_table + (size_t)s * a.pt_stride;
         const int pg0 = (k_begin + (int)(t * KT)) >> 4, pg_last = (k_end - 1) >> 4;      // 16-key pages (checked by the launcher)
         // pages past the last key are not looked up: the last valid one is loaded again (finite values, masked)
-        const int slot = pt[min(pg0 + (int)(lane & 7), pg_last)] * 16;
+        const int slot = max(0, pt[min(min(pg0 + (int)(lane & 7), pg_last), (int)a.pt_stride - 1)]) * 16;
         for (uint32_t gi = 0; gi < NG; ++gi) {
             const uint32_t g = NG > NB ? (gi == 0 ? NB : gi - 1) : gi, u0 = 2 * g, un = g < NB ? 2 : NU - 2 * NB;
             if (!__all_sync(0xffffffffu, mbar_wait_idle(bar_empty + 8 * g, (t & 1) ^ 1, abort_flag, 50))) return false;
@@ -268,8 +268,8 @@ latent_split_tc_kernel(QbLatent a, const __grid_constant__ CUtensorMap map, uint
 }
 
 struct MapKey {
-    int dev; const void *p; uint32_t pitch;
-    bool operator<(const MapKey &o) const { return std::tie(dev, p, pitch) < std::tie(o.dev, o.p, o.pitch); }
+    int dev; const void *p; uint64_t slots; uint32_t pitch;
+    bool operator<(const MapKey &o) const { return std::tie(dev, p, slots, pitch) < std::tie(o.dev, o.p, o.slots, o.pitch); }
 };
 std::map<MapKey, CUtensorMap> g_maps;
 std::mutex g_lock;
@@ -282,13 +282,12 @@ int launch(qb_ctx *ctx, const QbLatent &a, uint32_t n_splits, uint32_t NU, uint3
     {
         std::lock_guard<std::mutex> lock(g_lock);
         if (g_maps.size() > 4096) g_maps.clear();
-        const MapKey key{ctx->device, a.cache, a.pitch()};
+        const MapKey key{ctx->device, a.cache, a.slots, a.pitch()};
         auto it = g_maps.find(key);
         if (it == g_maps.end()) {
             CUtensorMap m;
-            // a box: one 128-byte column of a 16-key page.  The slot extent only bounds the coordinates TMA accepts; the kernel
-            // asks for pages of the page table alone.  Columns past the pitch read as zero.
-            QB_TRY(qb_make_tmap_2d(&m, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, a.cache, a.pitch(), 1ull << 30, (uint64_t)a.pitch() * 2, 64, 16, CU_TENSOR_MAP_SWIZZLE_128B));
+            // a box: one 128-byte column of a 16-key page; columns past the pitch read as zero
+            QB_TRY(qb_make_tmap_2d(&m, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, a.cache, a.pitch(), a.slots, (uint64_t)a.pitch() * 2, 64, 16, CU_TENSOR_MAP_SWIZZLE_128B));
             it = g_maps.emplace(key, m).first;
         }
         map = it->second;

@@ -66,7 +66,9 @@ struct QbLayerNorm {
     uint32_t vocab = 0;
     const float *parts = nullptr;             // [S][M][n]
     uint32_t S = 0;
-    const int32_t *row_map = nullptr;         // source rows of x (the stream is not written then)
+    const int32_t *row_map = nullptr;         // source rows of x (the stream is not written then), below x_rows
+    uint32_t x_rows = 0;
+    int *err_flag = nullptr;
     float *trace = nullptr;                   // copy of the residual before the loop's additions [M][n]
     float *emb_store = nullptr;               // the embedding output is kept here [M][n]
     const float *emb_add = nullptr;           // ... and added
@@ -107,7 +109,8 @@ struct QbLatent {
     const QbDense *ukv = nullptr;             // per head: dimp key rows, then vdimp value rows (rows past dim / vdim are zero)
     const int32_t *seq_pos = nullptr, *page_table = nullptr;
     uint32_t pt_stride = 0, page_size = 0, max_pos = 0;
-    void *cache = nullptr;                    // [slot][rankp + rotp], activation type
+    void *cache = nullptr;                    // [slots][rankp + rotp], activation type
+    uint64_t slots = 0;
     bool ingest = false;                      // a prompt chunk of one sequence
     uint32_t max_splits = 1;                  // spans a sequence's keys are cut into at most (absorbed form)
     // scratch (sizes: QbLatentScratch)
@@ -129,6 +132,15 @@ static const uint32_t QB_LAT_ABSORB_ROWS = 16;     // rows per sequence up to wh
 // Keys per span of a sequence's absorbed attention: its keys over at most max_splits spans of whole 64-key tiles.  A function
 // of the sequence's own length and of how many sequences share the launch; where the cuts fall changes rounding only.
 __device__ __forceinline__ uint32_t qb_latent_span(uint32_t keys, uint32_t max_splits) { return ((keys + max_splits - 1) / max_splits + 63) & ~63u; }
+#endif
+#ifdef __CUDACC__
+// Physical slot of a key of a sequence whose page-table row is pt, or -1 (an index past the row, an unassigned page).
+__device__ __forceinline__ int64_t qb_latent_slot(const QbLatent &a, const int32_t *pt, uint32_t key) {
+    const uint32_t i = key / a.page_size;
+    const int32_t page = i < a.pt_stride ? pt[i] : -1;
+    const int64_t slot = (int64_t)page * a.page_size + key % a.page_size;
+    return page >= 0 && (uint64_t)slot < a.slots ? slot : -1;
+}
 #endif
 // Whether prompt chunks of this shape expand keys and values (bfloat16, sizes within the kernel's registers).
 bool qb_latent_expands(const QbLatent &a);

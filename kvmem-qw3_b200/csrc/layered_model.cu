@@ -474,6 +474,7 @@ int latent_block(qb_ctx *ctx, qb_batch *b, uint32_t run, const RowSet &rs, uint3
     a.seq_pos = rs.seq_pos; a.max_pos = rs.max_pos; a.ingest = rs.ingest;
     a.page_table = b->page_table + (size_t)rs.seq0 * b->pages_per_seq; a.pt_stride = b->pages_per_seq; a.page_size = b->page_size;
     a.cache = B->cache[run];
+    a.slots = b->slots;
     a.max_splits = qb_latent_max_splits(a, rs.ns, (uint32_t)ctx->sm_count);
     a.q = B->q; a.qa = B->qa; a.part_acc = B->part_acc; a.part_ml = B->part_ml; a.lat = B->lat; a.kr = B->kr; a.kv = B->kv;
     a.out = B->mix;
@@ -534,7 +535,7 @@ int layered_head(qb_ctx *ctx, qb_batch *b, const int32_t *row_map, uint32_t rows
     QbLayeredBatch *B = b->layered;
     if (row_map) {
         QbLayerNorm n;
-        n.M = rows; n.n = Y.spec.width; n.eps = (float)Y.spec.eps; n.x = b->hid; n.row_map = row_map; n.w = Y.final_norm; n.out = B->x;
+        n.M = rows; n.n = Y.spec.width; n.eps = (float)Y.spec.eps; n.x = b->hid; n.x_rows = b->rows_cap + b->n_seqs; n.row_map = row_map; n.w = Y.final_norm; n.out = B->x;
         QB_TRY(qb_launch_layer_norm(ctx, n));
     }
     return qb_dense_gemm(ctx, Y.head, B->x, rows, dst, 1);

@@ -47,7 +47,11 @@ layer_norm_kernel(QbLayerNorm a) {
     QB_PDL_ENTER();
     __shared__ float red[LN_THREADS / 32];
     const uint32_t m = blockIdx.x, n = a.n, tid = threadIdx.x;
-    const uint32_t src = a.row_map ? (uint32_t)a.row_map[m] : m;
+    uint32_t src = a.row_map ? (uint32_t)a.row_map[m] : m;
+    if (a.row_map && src >= a.x_rows) {                                  // recorded, and row 0 read instead
+        if (tid == 0) atomicExch(a.err_flag, 6001);
+        src = 0;
+    }
     float *x = a.x + (size_t)src * n;
     Vec<V> row[NE];
     if (a.tokens) {
@@ -137,7 +141,9 @@ int launch(qb_ctx *ctx, const QbLayerNorm &a) {
 
 }  // namespace
 
-int qb_launch_layer_norm(qb_ctx *ctx, const QbLayerNorm &a) {
+int qb_launch_layer_norm(qb_ctx *ctx, const QbLayerNorm &args) {
+    QbLayerNorm a = args;
+    a.err_flag = ctx->err_flag_dev;
     QB_REQUIRE(a.M > 0, "layer norm: no rows");
     QB_REQUIRE(!a.w || (a.M <= a.out.cap && a.n <= a.out.ld), "layer norm: %u rows of %u elements exceed the output buffer", a.M, a.n);
     if (a.n % 4 == 0) return a.out.f32 ? launch<float, 4>(ctx, a) : launch<__nv_bfloat16, 4>(ctx, a);

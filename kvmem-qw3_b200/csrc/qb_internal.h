@@ -41,6 +41,7 @@ int qb_fail(int code, const char *fmt, ...);
         (ctx)->launches++;                                                                         \
         if ((ctx)->trace_on) qb_trace_mark(ctx, name);                                             \
         cudaError_t _e = cudaGetLastError();                                                       \
+        if (_e == cudaSuccess && (ctx)->sync_launches) _e = cudaStreamSynchronize((ctx)->stream);  \
         if (_e != cudaSuccess)                                                                     \
             return qb_fail(QB_ERR_CUDA, "launch of %s failed: %s", name, cudaGetErrorString(_e));  \
     } while (0)
@@ -77,6 +78,7 @@ struct qb_ctx {
     void *flush_buf = nullptr;             // > L2 bytes, written by qb_flush_l2
     size_t flush_bytes = 0;
     int *err_flag_dev = nullptr;           // set by kernels whose bounded waits ran out
+    bool sync_launches = false;            // QW3B200_SYNC_LAUNCHES=1: wait after every launch, so that an error names its kernel
     // optional launch trace (qb_trace_*): one event after every launch, durations = event deltas
     bool trace_on = false;
     std::vector<cudaEvent_t> trace_ev;
