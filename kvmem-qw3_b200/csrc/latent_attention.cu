@@ -217,6 +217,9 @@ __device__ __forceinline__ void ldsm2(uint32_t (&r)[2], uint32_t addr) {
 __device__ __forceinline__ void ldsm4t(uint32_t (&r)[4], uint32_t addr) {
     asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
 }
+__device__ __forceinline__ void ldsm2t(uint32_t (&r)[2], uint32_t addr) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x2.trans.shared.b16 {%0,%1}, [%2];" : "=r"(r[0]), "=r"(r[1]) : "r"(addr));
+}
 __device__ __forceinline__ void mma(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
     asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
                  : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
@@ -231,6 +234,129 @@ template <int N> __device__ __forceinline__ void cp_wait() { asm volatile("cp.as
 __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
     const __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
     return *reinterpret_cast<const uint32_t *>(&v);
+}
+
+// ---- the two per-head products for many rows (batched decode, bfloat16): 32 rows x 64 columns per CTA on mma.sync -------------
+// A warp takes 8 columns.  The weights are requested before the CTA waits for the kernel in front of it.
+constexpr uint32_t PR = 32, PC = 64;
+
+// qa[row][h] = [W_uk(h)^T q_n | q_r]: grid (H, latent columns / 64, rows / 32)
+__global__ void __launch_bounds__(LT)
+latent_absorb_mma_kernel(QbLatent a, const uint8_t *__restrict__ rec, uint32_t kc, uint32_t rows) {
+    asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
+    extern __shared__ __align__(16) uint8_t smem[];
+    const uint32_t h = blockIdx.x, c0 = blockIdx.y * PC, r0 = blockIdx.z * PR, tid = threadIdx.x, w = tid >> 5, lane = tid & 31;
+    const uint32_t dp = a.dimp(), per = dp + a.rotp(), rp = a.rankp(), D = a.pitch(), qp = (dp + 8) * 2, wp = (PC + 8) * 2;
+    const uint32_t qs = s32(smem), ws = qs + PR * qp;
+    for (uint32_t i = tid; i < dp * 8; i += LT)                         // [dp rows][64 columns]
+        cp16(ws + (i >> 3) * wp + (i & 7) * 16, rec + qb_dense_offset(kc, h * (dp + a.vdimp()) + (i >> 3), blockIdx.y * 8 + (i & 7)), true);
+    cp_commit();
+    asm volatile("griddepcontrol.wait;" ::: "memory");
+    const __nv_bfloat16 *q = (const __nv_bfloat16 *)a.q;
+    for (uint32_t i = tid; i < PR * (dp / 8); i += LT) {
+        const uint32_t r = i / (dp / 8), c = i % (dp / 8);
+        const bool ok = r0 + r < rows;
+        cp16(qs + r * qp + c * 16, ok ? q + ((size_t)(r0 + r) * a.H + h) * per + c * 8 : q, ok);
+    }
+    cp_commit();
+    cp_wait<0>();
+    __syncthreads();
+    float acc[2][4] = {};
+    for (uint32_t k = 0; k < dp / 16; ++k) {
+        uint32_t b[2];
+        ldsm2t(b, ws + (k * 16 + (lane & 15)) * wp + w * 16);
+#pragma unroll
+        for (int t = 0; t < 2; ++t) {
+            uint32_t f[4];
+            ldsm4(f, qs + (t * 16 + (lane & 15)) * qp + k * 32 + (lane >> 4) * 16);
+            mma(acc[t], f, b[0], b[1]);
+        }
+    }
+    __nv_bfloat16 *qa = (__nv_bfloat16 *)a.qa;
+#pragma unroll
+    for (int t = 0; t < 2; ++t)
+#pragma unroll
+        for (int i = 0; i < 4; i += 2) {
+            const uint32_t r = r0 + t * 16 + (lane >> 2) + (i >> 1) * 8, c = c0 + w * 8 + (lane & 3) * 2;
+            if (r < rows && c < rp)                                     // (weights past the latent are zero)
+                *reinterpret_cast<uint32_t *>(qa + ((size_t)r * a.H + h) * D + c) = pack_bf16(acc[t][i], acc[t][i + 1]);
+        }
+    if (blockIdx.y == 0)
+        for (uint32_t i = tid; i < PR * a.rotp(); i += LT) {
+            const uint32_t r = r0 + i / a.rotp(), j = i % a.rotp();
+            if (r < rows) qa[((size_t)r * a.H + h) * D + rp + j] = q[((size_t)r * a.H + h) * per + dp + j];
+        }
+}
+
+// Folds the spans, adds the sink, applies W_uv: grid (H, rows / 32, value dimensions / 64)
+__global__ void __launch_bounds__(LT)
+latent_merge_mma_kernel(QbLatent a, const uint8_t *__restrict__ rec, uint32_t kc, uint32_t rows, uint32_t n_splits) {
+    asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
+    extern __shared__ __align__(16) uint8_t smem[];
+    const uint32_t h = blockIdx.x, r0 = blockIdx.y * PR, v0 = blockIdx.z * PC, tid = threadIdx.x, w = tid >> 5, lane = tid & 31;
+    const uint32_t pitch = (kc * 64 + 8) * 2, vp = a.vdimp();
+    const uint32_t ls = s32(smem), ws = ls + PR * pitch;
+    float *wt = reinterpret_cast<float *>(smem + (PR + PC) * pitch);    // [32][n_splits]
+    __shared__ uint32_t cnt[PR];
+    for (uint32_t i = tid; i < PC * kc * 8; i += LT) {                  // [64 value rows][latent]
+        const uint32_t v = i / (kc * 8), c = i % (kc * 8);
+        const bool ok = v0 + v < vp;
+        cp16(ws + v * pitch + c * 16, rec + qb_dense_offset(kc, h * (a.dimp() + vp) + a.dimp() + (ok ? v0 + v : 0), c), ok);
+    }
+    cp_commit();
+    asm volatile("griddepcontrol.wait;" ::: "memory");
+    for (uint32_t j = w; j < PR; j += LT / 32) {
+        const uint32_t m = r0 + j;
+        uint32_t n = 0;
+        if (m < rows) {
+            const uint32_t base = (uint32_t)a.seq_pos[m / a.R], pos = base + m % a.R;
+            n = min(pos / qb_latent_span(base + a.R, a.max_splits) + 1, n_splits);
+            const float *ml = a.part_ml + ((size_t)m * a.H + h) * n_splits * 2;
+            const float sink = a.sink[h];
+            float mx = sink;
+            for (uint32_t i = lane; i < n; i += 32) mx = fmaxf(mx, ml[2 * i]);
+            mx = warp_max(mx);
+            float den = 0.0f;
+            for (uint32_t i = lane; i < n; i += 32) den += ml[2 * i + 1] * expf(ml[2 * i] - mx);
+            den = warp_sum(den) + expf(sink - mx);
+            for (uint32_t i = lane; i < n; i += 32) wt[j * n_splits + i] = expf(ml[2 * i] - mx) / den;
+        }
+        if (lane == 0) cnt[j] = n;
+    }
+    __syncthreads();
+    const uint32_t half = kc * 32;                                      // column pairs
+#pragma unroll 4
+    for (uint32_t t = tid; t < PR * half; t += LT) {
+        const uint32_t r = t / half, c = (t % half) * 2, n = cnt[r];
+        const float *acc = a.part_acc + ((size_t)(r0 + r) * a.H + h) * n_splits * a.rank + c;
+        float x = 0.0f, y = 0.0f;
+        for (uint32_t i = 0; i < n; ++i) {
+            const float f = wt[r * n_splits + i];
+            if (c < a.rank) x = fmaf(f, acc[(size_t)i * a.rank], x);
+            if (c + 1 < a.rank) y = fmaf(f, acc[(size_t)i * a.rank + 1], y);
+        }
+        *reinterpret_cast<uint32_t *>(smem + r * pitch + c * 2) = pack_bf16(x, y);
+    }
+    cp_wait<0>();
+    __syncthreads();
+    float acc[2][4] = {};
+    for (uint32_t k = 0; k < kc * 4; ++k) {
+        uint32_t b[2];
+        ldsm2(b, ws + (w * 8 + (lane & 7)) * pitch + k * 32 + ((lane >> 3) & 1) * 16);
+#pragma unroll
+        for (int t = 0; t < 2; ++t) {
+            uint32_t f[4];
+            ldsm4(f, ls + (t * 16 + (lane & 15)) * pitch + k * 32 + (lane >> 4) * 16);
+            mma(acc[t], f, b[0], b[1]);
+        }
+    }
+#pragma unroll
+    for (int t = 0; t < 2; ++t)
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            const uint32_t r = r0 + t * 16 + (lane >> 2) + (i >> 1) * 8, v = v0 + w * 8 + (lane & 3) * 2 + (i & 1);
+            if (r < rows && v < a.vdim) ((__nv_bfloat16 *)a.out.p + (size_t)r * a.out.ld + h * a.vdim)[v] = __float2bfloat16(acc[t][i]);
+        }
 }
 
 // ---- absorbed attention on mma.sync: 16 MT queries per CTA over one span of keys, 64-key tiles --------------------------------
@@ -674,7 +800,7 @@ int launch_merge(qb_ctx *ctx, const QbLatent &a, uint32_t rows, uint32_t n_split
     const size_t smem = (((size_t)MB * n_splits + 3) / 4 * 4 + MB * kc * 64) * sizeof(float);
     QB_REQUIRE(smem <= 227 * 1024, "latent attention: a latent of %u does not fit", a.rank);
     QB_CUDA(cudaFuncSetAttribute(latent_merge_kernel<T, MB>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-    const uint32_t vz = std::max(1u, std::min((a.vdim + 31) / 32, (4u * (uint32_t)ctx->sm_count + a.H * groups - 1) / (a.H * groups)));
+    const uint32_t vz = std::max(1u, std::min((a.vdim + 31) / 32, (2u * (uint32_t)ctx->sm_count) / (a.H * groups)));
     QB_CUDA(qb_launch_pdl(ctx->stream, latent_merge_kernel<T, MB>, dim3(a.H, groups, vz), dim3(LT), smem, a, (const uint8_t *)a.ukv->rec, kc, rows, n_splits));
     QB_LAUNCHED(ctx, "latent_merge_kernel");
     return QB_OK;
@@ -685,7 +811,15 @@ int latent_absorbed(qb_ctx *ctx, QbLatent a) {
     const uint32_t rows = a.ns * a.R;
     if (a.R > QB_LAT_ABSORB_ROWS) a.max_splits = 1;          // the rows alone fill the GPU
     const uint32_t n_splits = std::min(a.max_splits, (a.max_pos + 63) / 64);
-    if (rows == 1) QB_TRY((launch_absorb<T, 1>(ctx, a, rows)));
+    const size_t sm_ab = (size_t)PR * (a.dimp() + 8) * 2 + (size_t)a.dimp() * (PC + 8) * 2;
+    const size_t sm_me = (size_t)(PR + PC) * (a.ukv->kc * 64 + 8) * 2 + (size_t)PR * n_splits * sizeof(float);
+    const bool many = !a.f32 && rows >= 8 && sm_ab <= 200 * 1024 && sm_me <= 200 * 1024;
+    if (many) {
+        QB_CUDA(cudaFuncSetAttribute(latent_absorb_mma_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sm_ab));
+        QB_CUDA(qb_launch_pdl(ctx->stream, latent_absorb_mma_kernel, dim3(a.H, (a.rankp() + PC - 1) / PC, (rows + PR - 1) / PR), dim3(LT), sm_ab, a,
+                              (const uint8_t *)a.ukv->rec, a.ukv->kc, rows));
+        QB_LAUNCHED(ctx, "latent_absorb_mma_kernel");
+    } else if (rows == 1) QB_TRY((launch_absorb<T, 1>(ctx, a, rows)));
     else QB_TRY((launch_absorb<T, 8>(ctx, a, rows)));
     const uint32_t MT = a.R * a.H > 16 ? 2 : 1;
     static const bool use_tc = qb_env_u32("QW3B200_LATENT_TC", 1) != 0;       // 0: the mma.sync form, for comparison
@@ -696,6 +830,13 @@ int latent_absorbed(qb_ctx *ctx, QbLatent a) {
         else QB_TRY(launch_split_nv<1>(ctx, a, n_splits));
     } else {
         QB_TRY(launch_simt<T>(ctx, a, n_splits));
+    }
+    if (many) {
+        QB_CUDA(cudaFuncSetAttribute(latent_merge_mma_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sm_me));
+        QB_CUDA(qb_launch_pdl(ctx->stream, latent_merge_mma_kernel, dim3(a.H, (rows + PR - 1) / PR, (a.vdimp() + PC - 1) / PC), dim3(LT), sm_me, a,
+                              (const uint8_t *)a.ukv->rec, a.ukv->kc, rows, n_splits));
+        QB_LAUNCHED(ctx, "latent_merge_mma_kernel");
+        return QB_OK;
     }
     if (rows == 1) return launch_merge<T, 1>(ctx, a, rows, n_splits);
     return launch_merge<T, 4>(ctx, a, rows, n_splits);

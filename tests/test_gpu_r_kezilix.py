@@ -254,6 +254,26 @@ def test_unequal_batch_equals_each_alone(make, dtype):
     b.close()
 
 
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_large_batch(make, dtype):
+    """34 sequences decoded together (more than one 32-row block of the per-head products), then the first 9 of them."""
+    c = make(MIXED)
+    n = 34
+    prompts = [c.tokens(1 + (37 * s) % 140) for s in range(n)]
+    b = c.batch(dtype, n_seqs=n, max_ctx=160, pool_pages=10 * n)
+    for s, p in enumerate(prompts):
+        b.prefill(s, p)
+    seqs = [p + t for p, t in zip(prompts, b.read_output())]
+    for active in (n, n, 9):
+        b.set_active(active)
+        b.greedy_step()
+        got = b.last_logits(active)
+        close_to(got, np.stack([c.want(seqs[s])[-1] for s in range(active)]), dtype, "%d active" % active)
+        for s, t in enumerate(b.read_output()[:active]):
+            seqs[s] = seqs[s] + t
+    b.close()
+
+
 def test_pages_and_slots_used_again(make):
     """Requests interleaved over a small pool: slots and pages return with other contents."""
     c = make(MIXED)
