@@ -134,6 +134,9 @@ ALONE = {
     "loop_from_first": config([ret(), lat()], loop={"start": 0, "stop": 1, "times": 3}),
     "loop_to_last": config([ret(), ret(), lat()], loop={"start": 1, "stop": 3, "times": 4}),
     "loop_once": config([ret(), lat(), ret()], loop={"start": 1, "stop": 2, "times": 1}),
+    "odd_width": config([ret(heads=3, dim=22, vdim=30, rot=10, ff=33), lat(heads=3, dim=18, rot_dim=6, rot=6, vdim=17, rank=45, ff=50)], width=90, vocab=131),
+    "odd_width_prime": config([lat(heads=1, dim=7, rot_dim=2, rot=2, vdim=5, rank=19, ff=11), ret(heads=1, dim=3, vdim=7, rot=2, decay=(0.9,))], width=67, vocab=101,
+                              loop={"start": 0, "stop": 2, "times": 2}),
     "mixed": MIXED,
 }
 
