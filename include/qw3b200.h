@@ -316,8 +316,8 @@ int  qb_model_load_gguf(qb_ctx *ctx, const char *path, qb_model **out, qb_model_
 int  qb_gguf_read_config(const char *path, qb_model_config *cfg_out, uint64_t *n_tensors_out, uint64_t *tensor_bytes_out);
 const qb_model_config *qb_model_get_config(const qb_model *m);
 /* A model by path: a GGUF file (qwen35), or a folder with config.json and model.safetensors whose config.json names an
- * architecture of the loader table ("Kezilix": a layered model -- retention and latent-attention layers, dense
- * feed-forwards, a looped span -- with bfloat16 weights).  f32 != 0: every product and activation in 32 bits (layered
+ * architecture of the loader table ("Kezilix", "Figonex": layered models -- recurrent and attention layers, dense
+ * feed-forwards, looped spans, shared layer weights -- with bfloat16 weights).  f32 != 0: every product and activation in 32 bits (layered
  * models only, QB_ERR_UNSUPPORTED otherwise).  cfg_out (may be NULL): of a layered model, only n_layers, n_embd,
  * vocab_size and rms_eps are set. */
 int  qb_model_load(qb_ctx *ctx, const char *path, int f32, qb_model **out, qb_model_config *cfg_out);

@@ -1746,6 +1746,7 @@ extern "C" int qb_debug_last_drafts(qb_ctx *ctx, qb_batch *b, int32_t *host_out)
 // ---- model folders: config.json names the architecture -----------------------------------------------------------------
 static const QbLoader LOADERS[] = {
     {"Kezilix", qb_layered_load},
+    {"Figonex", qb_layered_load},
 };
 
 extern "C" int qb_model_load(qb_ctx *ctx, const char *path, int f32, qb_model **out, qb_model_config *cfg_out) {

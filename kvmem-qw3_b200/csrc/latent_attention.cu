@@ -145,15 +145,15 @@ latent_split_simt_kernel(QbLatent a, uint32_t n_splits) {
     extern __shared__ float sm[];
     const uint32_t D = a.pitch(), DP = D + 1, tid = threadIdx.x, w = tid >> 5, lane = tid & 31;
     float *qs = sm, *ts = qs + SQ * D, *pr = ts + SK * DP, *al = pr + SQ * SK;
-    const uint32_t split = blockIdx.x, s = blockIdx.z, nq = a.R * a.H, q0 = blockIdx.y * SQ;
+    const uint32_t split = blockIdx.x, sg = blockIdx.z, s = sg / a.groups, grp = sg % a.groups, hg = a.heads_per_group(), nq = a.R * hg, q0 = blockIdx.y * SQ;
     const int base = a.seq_pos[s];
     const uint32_t span = qb_latent_span((uint32_t)base + a.R, a.max_splits);
     const uint32_t q_last = min(q0 + SQ, nq) - 1;
-    const int k_begin = (int)(split * span), k_end = min(k_begin + (int)span, base + (int)(q_last / a.H) + 1);
+    const int k_begin = (int)(split * span), k_end = min(k_begin + (int)span, base + (int)(q_last / hg) + 1);
     if (k_begin >= k_end) return;
-    const T *qa = (const T *)a.qa + ((size_t)s * nq + q0) * D;
+    const T *qa = (const T *)a.qa + ((size_t)sg * nq + q0) * D;
     for (uint32_t i = tid; i < SQ * D; i += LT) qs[i] = q0 + i / D < nq ? qb_f32(qa[i]) : 0.0f;
-    const int my_pos = q0 + w < nq ? base + (int)((q0 + w) / a.H) : -1;
+    const int my_pos = q0 + w < nq ? base + (int)((q0 + w) / hg) : -1;
     const int32_t *pt = a.page_table + (size_t)s * a.pt_stride;
     float mx = -INFINITY, sum = 0.0f, acc[SQ][SCOLS] = {};
     for (int kt = k_begin; kt < k_end; kt += SK) {
@@ -163,13 +163,17 @@ latent_split_simt_kernel(QbLatent a, uint32_t n_splits) {
             const int key = kt + (int)j;
             float v = 0.0f;
             const int64_t at = key < k_end ? qb_latent_slot(a, pt, (uint32_t)key) : -1;
-            if (at >= 0) v = qb_f32(((const T *)a.cache)[(size_t)at * D + e]);
+            if (at >= 0) v = qb_f32(((const T *)a.cache)[((size_t)at * a.groups + grp) * D + e]);
             ts[j * DP + e] = v;
         }
         __syncthreads();
         float sc = 0.0f;
         for (uint32_t e = 0; e < D; ++e) sc = fmaf(qs[w * D + e], ts[lane * DP + e], sc);
         const int key = kt + (int)lane;
+        if (a.key_scale && key < k_end) {
+            const int64_t at = qb_latent_slot(a, pt, (uint32_t)key);
+            sc *= at >= 0 ? a.key_scale[(size_t)at * a.groups + grp] : 0.0f;
+        }
         sc = key <= my_pos && key < k_end ? sc * a.scale : -INFINITY;
         const float nm = fmaxf(mx, warp_max(sc));
         const float p = sc == -INFINITY ? 0.0f : expf(sc - nm), alpha = mx == -INFINITY ? 0.0f : expf(mx - nm);
@@ -193,14 +197,14 @@ latent_split_simt_kernel(QbLatent a, uint32_t n_splits) {
         }
     }
     if (lane == 0 && q0 + w < nq) {
-        float *ml = a.part_ml + (((size_t)s * nq + q0 + w) * n_splits + split) * 2;
+        float *ml = a.part_ml + (((size_t)sg * nq + q0 + w) * n_splits + split) * 2;
         ml[0] = mx;
         ml[1] = sum;
     }
 #pragma unroll
     for (int q = 0; q < SQ; ++q)
         if (q0 + q < nq) {
-            float *dst = a.part_acc + (((size_t)s * nq + q0 + q) * n_splits + split) * a.rank;
+            float *dst = a.part_acc + (((size_t)sg * nq + q0 + q) * n_splits + split) * a.rank;
 #pragma unroll
             for (int i = 0; i < SCOLS; ++i) if (tid + i * LT < a.rank) dst[tid + i * LT] = acc[q][i];
         }
@@ -779,7 +783,7 @@ int launch_simt(qb_ctx *ctx, const QbLatent &a, uint32_t n_splits) {
     const size_t smem = ((size_t)SQ * D + SK * (D + 1) + SQ * SK + SQ) * sizeof(float);
     QB_REQUIRE(smem <= 227 * 1024 && a.rank <= SCOLS * LT, "latent attention: a latent of %u + %u does not fit", a.rank, a.rot_dim);
     QB_CUDA(cudaFuncSetAttribute(latent_split_simt_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-    QB_CUDA(qb_launch_pdl(ctx->stream, latent_split_simt_kernel<T>, dim3(n_splits, (a.R * a.H + SQ - 1) / SQ, a.ns), dim3(LT), smem, a, n_splits));
+    QB_CUDA(qb_launch_pdl(ctx->stream, latent_split_simt_kernel<T>, dim3(n_splits, (a.group_queries() + SQ - 1) / SQ, a.ns * a.groups), dim3(LT), smem, a, n_splits));
     QB_LAUNCHED(ctx, "latent_split_simt_kernel");
     return QB_OK;
 }
@@ -847,6 +851,10 @@ int latent_absorbed(qb_ctx *ctx, QbLatent a) {
 uint32_t qb_latent_max_splits(const QbLatent &a, uint32_t ns, uint32_t sms) {
     const uint32_t groups = (a.H + 47) / 48;
     return std::max(1u, std::min(64u, sms / (ns * groups)));
+}
+
+int qb_launch_latent_split_simt(qb_ctx *ctx, const QbLatent &a, uint32_t n_splits) {
+    return a.f32 ? launch_simt<float>(ctx, a, n_splits) : launch_simt<__nv_bfloat16>(ctx, a, n_splits);
 }
 
 bool qb_latent_expands(const QbLatent &a) {

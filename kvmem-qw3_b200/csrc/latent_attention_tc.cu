@@ -84,11 +84,11 @@ latent_split_tc_kernel(QbLatent a, const __grid_constant__ CUtensorMap map, uint
     asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
     asm volatile("griddepcontrol.wait;" ::: "memory");
 
-    const uint32_t split = blockIdx.x, s = blockIdx.z, nq = a.R * a.H, qg = blockIdx.y * NQ;
+    const uint32_t split = blockIdx.x, sg = blockIdx.z, s = sg / a.groups, grp = sg % a.groups, hg = a.heads_per_group(), nq = a.R * hg, qg = blockIdx.y * NQ;
     const int base = a.seq_pos[s];
     const uint32_t span = qb_latent_span((uint32_t)base + a.R, a.max_splits);
     const uint32_t q_last = min(qg + NQ, nq) - 1;
-    const int k_begin = (int)(split * span), k_end = min(k_begin + (int)span, base + (int)(q_last / a.H) + 1);
+    const int k_begin = (int)(split * span), k_end = min(k_begin + (int)span, base + (int)(q_last / hg) + 1);
     const uint32_t n_tiles = k_begin < k_end ? (uint32_t)(k_end - k_begin + KT - 1) / KT : 0;      // 0: nothing visible (uniform)
     // Loads of tile t: lane & 7 names a page of the tile, `slot` its first slot.
     auto load_tile = [&](uint32_t t) -> bool {
@@ -104,7 +104,7 @@ latent_split_tc_kernel(QbLatent a, const __grid_constant__ CUtensorMap map, uint
             __syncwarp();
             for (uint32_t i = lane; i < un * 8; i += 32) {               // (i & 7 == lane & 7)
                 const uint32_t u = u0 + (i >> 3);
-                tma_load_2d(smem_u32(smem + u * UNIT) + (i & 7) * 2048, &map, (int)(u * 64), slot, full);
+                tma_load_2d(smem_u32(smem + u * UNIT) + (i & 7) * 2048, &map, (int)(grp * a.pitch() + u * 64), slot, full);
             }
         }
         return true;
@@ -113,14 +113,14 @@ latent_split_tc_kernel(QbLatent a, const __grid_constant__ CUtensorMap map, uint
     if (n_tiles) {
         // queries in the swizzled K-major operand layout: [unit][NQ rows][128 B]; columns past the pitch and rows past the last query zero
         const uint32_t D = a.pitch();
-        const __nv_bfloat16 *qa = (const __nv_bfloat16 *)a.qa + ((size_t)s * nq + qg) * D;
+        const __nv_bfloat16 *qa = (const __nv_bfloat16 *)a.qa + ((size_t)sg * nq + qg) * D;
         for (uint32_t i = tid; i < NQ * NU * 8; i += C::THREADS) {
             const uint32_t q = i / (NU * 8), c8 = i % (NU * 8);
             uint4 v = make_uint4(0u, 0u, 0u, 0u);
             if (qg + q < nq && c8 * 8 < D) v = *reinterpret_cast<const uint4 *>(qa + (size_t)q * D + c8 * 8);
             *reinterpret_cast<uint4 *>(smem + L.q + (c8 >> 3) * (NQ * 128) + q * 128 + (((c8 & 7) ^ (q & 7)) << 4)) = v;
         }
-        if (tid < NQ) qpos[tid] = qg + tid < nq ? base + (int)((qg + tid) / a.H) : -1;
+        if (tid < NQ) qpos[tid] = qg + tid < nq ? base + (int)((qg + tid) / hg) : -1;
         asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
     }
     tc_fence_before();
@@ -168,7 +168,15 @@ latent_split_tc_kernel(QbLatent a, const __grid_constant__ CUtensorMap map, uint
     } else {
         const uint32_t quarter = warp & 3, q0 = ((warp - 2) >> 2) * 16, r = quarter * 32 + lane;      // key lane, first query column
         const uint32_t lane_addr = (quarter * 32u) << 16;
-        const float sl = a.scale * LOG2E;
+        // factor of a key's scores, looked up a tile ahead
+        const float sl0 = a.scale * LOG2E;
+        auto key_factor = [&](uint32_t t) -> float {
+            const int key = k_begin + (int)(t * KT + r);
+            if (!a.key_scale || key >= k_end) return sl0;
+            const int64_t at = qb_latent_slot(a, a.page_table + (size_t)s * a.pt_stride, (uint32_t)key);
+            return at < 0 ? 0.0f : sl0 * a.key_scale[(size_t)at * a.groups + grp];
+        };
+        float sl_next = key_factor(0);
         const float4 *red4 = reinterpret_cast<const float4 *>(red);
         uint8_t *prow = smem + L.p + (r >> 6) * (NQ * 128) + (r & 7) * 2;
         const uint32_t ch = (r & 63) >> 3;
@@ -185,6 +193,8 @@ latent_split_tc_kernel(QbLatent a, const __grid_constant__ CUtensorMap map, uint
             tmem_ld16(tmem_s + lane_addr + q0, raw);
             tmem_wait_dep(raw);
             const int key = k_begin + (int)(t * KT + r);
+            const float sl = sl_next;
+            if (t + 1 < n_tiles) sl_next = key_factor(t + 1);
             float sc[16], cm[16];
 #pragma unroll
             for (int j = 0; j < 16; ++j) {
@@ -233,7 +243,7 @@ latent_split_tc_kernel(QbLatent a, const __grid_constant__ CUtensorMap map, uint
         if (lane < 16) red[(rb + q0 + lane) * 4 + quarter] = wsum;
         asm volatile("bar.sync %0, 128;" ::"r"(1 + q0 / 16) : "memory");
         if (ok) {
-            const size_t row0 = (size_t)s * nq + qg + q0;
+            const size_t row0 = (size_t)sg * nq + qg + q0;
             if (quarter == 0 && lane < 16 && qg + q0 + lane < nq) {
                 const float4 l4 = red4[rb + q0 + lane];
                 float m = mx[0];
@@ -268,8 +278,8 @@ latent_split_tc_kernel(QbLatent a, const __grid_constant__ CUtensorMap map, uint
 }
 
 struct MapKey {
-    int dev; const void *p; uint64_t slots; uint32_t pitch;
-    bool operator<(const MapKey &o) const { return std::tie(dev, p, slots, pitch) < std::tie(o.dev, o.p, o.slots, o.pitch); }
+    int dev; const void *p; uint64_t slots; uint32_t cols;
+    bool operator<(const MapKey &o) const { return std::tie(dev, p, slots, cols) < std::tie(o.dev, o.p, o.slots, o.cols); }
 };
 std::map<MapKey, CUtensorMap> g_maps;
 std::mutex g_lock;
@@ -282,26 +292,31 @@ int launch(qb_ctx *ctx, const QbLatent &a, uint32_t n_splits, uint32_t NU, uint3
     {
         std::lock_guard<std::mutex> lock(g_lock);
         if (g_maps.size() > 4096) g_maps.clear();
-        const MapKey key{ctx->device, a.cache, a.slots, a.pitch()};
+        const uint32_t cols = a.groups * a.pitch();
+        const MapKey key{ctx->device, a.cache, a.slots, cols};
         auto it = g_maps.find(key);
         if (it == g_maps.end()) {
             CUtensorMap m;
-            // a box: one 128-byte column of a 16-key page; columns past the pitch read as zero
-            QB_TRY(qb_make_tmap_2d(&m, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, a.cache, a.pitch(), a.slots, (uint64_t)a.pitch() * 2, 64, 16, CU_TENSOR_MAP_SWIZZLE_128B));
+            // a box: one 128-byte column of a 16-key page; columns past a vector read as the next group's (their queries are zero),
+            // past the last as zero
+            QB_TRY(qb_make_tmap_2d(&m, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, a.cache, cols, a.slots, (uint64_t)cols * 2, 64, 16, CU_TENSOR_MAP_SWIZZLE_128B));
             it = g_maps.emplace(key, m).first;
         }
         map = it->second;
     }
-    QB_CUDA(qb_launch_pdl(ctx->stream, latent_split_tc_kernel<NQ>, dim3(n_splits, (a.R * a.H + NQ - 1) / NQ, a.ns), dim3(LtcCfg<NQ>::THREADS), (size_t)smem, a, map,
+    QB_CUDA(qb_launch_pdl(ctx->stream, latent_split_tc_kernel<NQ>, dim3(n_splits, (a.group_queries() + NQ - 1) / NQ, a.ns * a.groups), dim3(LtcCfg<NQ>::THREADS), (size_t)smem, a, map,
                           n_splits, NU, NB));
     QB_LAUNCHED(ctx, "latent_split_tc_kernel");
     return QB_OK;
 }
 
+// 64-column units of a tile (the latent columns go in pairs; a unit past the vector holds columns nobody uses).
+uint32_t units_of(const QbLatent &a) { return std::max((a.pitch() + 63) / 64, (a.rankp() + 127) / 128 * 2); }
+
 // Queries per CTA: the fewest groups, then the smallest tile; 0 when the shape does not fit.
 uint32_t pick_nq(const QbLatent &a) {
-    const uint32_t NU = (a.pitch() + 63) / 64, NB = (a.rankp() + 127) / 128, nq = a.R * a.H;
-    if (a.f32 || a.page_size != 16 || NB > 4 || 2 * NB > NU) return 0;
+    const uint32_t NU = units_of(a), NB = (a.rankp() + 127) / 128, nq = a.group_queries();
+    if (a.f32 || a.page_size != 16 || NB > 4) return 0;
     uint32_t best = 0;
     for (uint32_t n : {16u, 32u, 48u}) {
         if (ltc_smem(NU, n).total > 232448) continue;
@@ -315,7 +330,7 @@ uint32_t pick_nq(const QbLatent &a) {
 bool qb_latent_tc_supports(const QbLatent &a) { return pick_nq(a) != 0; }
 
 int qb_launch_latent_split_tc(qb_ctx *ctx, const QbLatent &a, uint32_t n_splits) {
-    const uint32_t NU = (a.pitch() + 63) / 64, NB = (a.rankp() + 127) / 128;
+    const uint32_t NU = units_of(a), NB = (a.rankp() + 127) / 128;
     switch (pick_nq(a)) {
         case 16: return launch<16>(ctx, a, n_splits, NU, NB);
         case 32: return launch<32>(ctx, a, n_splits, NU, NB);

@@ -1,6 +1,7 @@
 // Layered models: decoders described layer by layer in a config.json (mixer type and sizes, feed-forward, an optional loop
-// over a span of layers), with dense bfloat16 weights.  Mechanisms (retention.cu, latent_attention.cu, dense_gemm.cu,
-// layered_norm.cu) take their constants as arguments; layered_model.cu composes them.
+// over a span of layers, layers that share weights), with dense bfloat16 weights.  Mechanisms (linear_recurrence.cu,
+// latent_attention.cu, shared_kv_attention.cu, dense_gemm.cu, layered_norm.cu) take their constants as arguments;
+// layered_model.cu composes them.
 #pragma once
 
 #include "dense_gemm.h"
@@ -20,6 +21,7 @@ template <> __device__ __forceinline__ float qb_cast<float>(float v) { return v;
 template <> __device__ __forceinline__ __nv_bfloat16 qb_cast<__nv_bfloat16>(float v) { return __float2bfloat16(v); }
 __device__ __forceinline__ float qb_f32(float v) { return v; }
 __device__ __forceinline__ float qb_f32(__nv_bfloat16 v) { return __bfloat162float(v); }
+__device__ __forceinline__ float qb_sigmoid(float z) { return __fdiv_rn(1.0f, 1.0f + expf(-z)); }
 // 32-bit angles: cos and sin of pair i at a position
 __device__ __forceinline__ void qb_rot_angle(const QbRotary &r, int pos, uint32_t i, float &c, float &s) {
     sincosf((float)pos * r.freq[i], &s, &c);
@@ -58,14 +60,20 @@ __device__ __forceinline__ float qb_block_sum(float v, float *red, uint32_t nwar
 struct QbLayerNorm {
     uint32_t M = 0, n = 0;
     float eps = 0.0f;
+    bool center = false;                      // layer norms (mean off first), else RMS norms
     float *x = nullptr;                       // residual stream [M][n]
-    // source of the row: an embedding row (normalised with embed_w), or x + sum of parts
+    // source of the row: an embedding row (scaled; normalised with embed_w where given), or x + sum of parts (the sum normalised
+    // with post_w where given)
     const int32_t *tokens = nullptr;
     const __nv_bfloat16 *embed = nullptr;     // [vocab][n]
     const float *embed_w = nullptr;
+    float embed_scale = 1.0f;
     uint32_t vocab = 0;
     const float *parts = nullptr;             // [S][M][n]
     uint32_t S = 0;
+    const float *row_ss = nullptr;            // sums of squares [M][ss_n] of ss_len elements: the sum of parts is divided by their
+    uint32_t ss_n = 0, ss_len = 0;            // root mean square first (a norm that commutes with the product)
+    const float *post_w = nullptr;            // norm on the sublayer's result, gain [n]
     const int32_t *row_map = nullptr;         // source rows of x (the stream is not written then), below x_rows
     uint32_t x_rows = 0;
     int *err_flag = nullptr;
@@ -73,27 +81,47 @@ struct QbLayerNorm {
     float *emb_store = nullptr;               // the embedding output is kept here [M][n]
     const float *emb_add = nullptr;           // ... and added
     const float *step = nullptr;              // vector [n] added to every row
-    const float *w = nullptr;                 // gain of the norm that follows; null: no output
+    const float *w = nullptr;                 // gain of the norm that follows; null: the row goes out as it is
     QbActBuf out;
 };
 int qb_launch_layer_norm(qb_ctx *ctx, const QbLayerNorm &a);
 
-// ---- retention (retention.cu) -------------------------------------------------------------------------------------------
-// Linear attention with one fixed decay per head: S_t = decay S_(t-1) + k_t v_t^T, o_t = S_t^T q_t, o divided by its root
-// mean square and gated by silu(g).  Rows are grouped per sequence (R rows each, consecutive positions).
-static const uint32_t QB_RET_CHUNK = 64;
-struct QbRetention {
-    float *proj = nullptr;                    // [S][rows][stride]: q (H*dim) | k (H*dim) | v (H*vdim) | g (H*vdim)
+// ---- linear recurrences (linear_recurrence.cu) ---------------------------------------------------------------------------
+// A matrix state per head, S_t = decay S_(t-1) + k_t v_t^T, o_t = S_t^T q_t, normalised and gated.  Rows are grouped per
+// sequence (R rows each, consecutive positions).
+static const uint32_t QB_REC_CHUNK = 64, QB_REC_SLICE = 32;
+struct QbRecurrence {
+    float *proj = nullptr;                    // [S][rows][stride]: q (H*dim) | k (H*dim) | v (H*vdim) | g (H*vdim) | gated: i (H) | f (H)
     uint32_t S = 1, stride = 0;
     uint32_t ns = 0, R = 0, H = 0, dim = 0, vdim = 0;
     float eps = 0.0f;
-    QbRotary rot;
-    const float *powers = nullptr;            // [H][QB_RET_CHUNK + 1]: decay^0 .. decay^64
+    QbRotary rot;                             // of q and k
+    bool act = false;                         // silu on q, k and v
+    float qscale = 1.0f, kscale = 1.0f;
+    bool sigmoid_gate = false;                // the output's gate: sigmoid(g), else silu(g)
+    const float *norm_w = nullptr;            // [H*vdim] weight of the output's norm, or none
+    // The output's norm is per head, or (row_ss set) spans all heads: the rows go out without it, and their sums of squares
+    // [rows][H] go to the consumer of the output projection, which scales its rows.
+    float *row_ss = nullptr;
+    const float *powers = nullptr;            // fixed decays: [H][QB_REC_CHUNK + 1]: decay^0 .. decay^64
+    // gated: log gates cap * tanh((z + bias) / cap) per token and head (the forget gate through a log sigmoid), running maximum,
+    // normaliser
+    bool gated = false;
+    const float *i_bias = nullptr, *f_bias = nullptr;
+    float cap = 1.0f;
+    float *row_aux = nullptr;                 // scratch [rows][H][2]
     const int32_t *seq_pos = nullptr;
-    float *state = nullptr;                   // [ns][H][dim][vdim]
+    float *state = nullptr;                   // [ns][state_stride]
+    size_t state_stride = 0;
     QbActBuf out;                             // [rows][H*vdim]
 };
-int qb_launch_retention(qb_ctx *ctx, const QbRetention &a);
+__host__ __device__ inline uint32_t qb_recurrence_slices(uint32_t vdim) { return (vdim + QB_REC_SLICE - 1) / QB_REC_SLICE; }
+// Floats of one sequence's state: [H][dim][vdim]; gated: also n [H][dim] and m [H][slices].
+inline size_t qb_recurrence_state(uint32_t H, uint32_t dim, uint32_t vdim, bool gated) {
+    const size_t n = (size_t)H * dim * vdim + (gated ? (size_t)H * (dim + qb_recurrence_slices(vdim)) : 0);
+    return (n + 3) & ~(size_t)3;
+}
+int qb_launch_recurrence(qb_ctx *ctx, const QbRecurrence &a);
 
 // ---- latent attention (latent_attention.cu) ----------------------------------------------------------------------------
 // Keys and values of all heads come from one latent vector per token; the cache holds the latent and one rotated key part
@@ -109,7 +137,12 @@ struct QbLatent {
     const QbDense *ukv = nullptr;             // per head: dimp key rows, then vdimp value rows (rows past dim / vdim are zero)
     const int32_t *seq_pos = nullptr, *page_table = nullptr;
     uint32_t pt_stride = 0, page_size = 0, max_pos = 0;
-    void *cache = nullptr;                    // [slots][rankp + rotp], activation type
+    void *cache = nullptr;                    // [slots][groups][rankp + rotp], activation type
+    // Key/value groups: `groups` cached vectors per token, each attended by H / groups consecutive heads (latent attention: one,
+    // by all); key_scale [slots][groups]: a factor of a vector's scores.  Queries qa and spans lie group by group:
+    // [sequence][group][row][head of the group].
+    uint32_t groups = 1;
+    const float *key_scale = nullptr;
     uint64_t slots = 0;
     bool ingest = false;                      // a prompt chunk of one sequence
     uint32_t max_splits = 1;                  // spans a sequence's keys are cut into at most (absorbed form)
@@ -126,6 +159,8 @@ struct QbLatent {
     __host__ __device__ uint32_t vdimp() const { return (vdim + 15) & ~15u; }
     __host__ __device__ uint32_t rankp() const { return (rank + 15) & ~15u; }
     __host__ __device__ uint32_t pitch() const { return rankp() + rotp(); }
+    __host__ __device__ uint32_t heads_per_group() const { return H / groups; }
+    __host__ __device__ uint32_t group_queries() const { return R * heads_per_group(); }
 };
 static const uint32_t QB_LAT_ABSORB_ROWS = 16;     // rows per sequence up to which the absorbed form runs
 #ifdef __CUDACC__
@@ -147,8 +182,27 @@ bool qb_latent_expands(const QbLatent &a);
 // The absorbed form's spans on tcgen05 (latent_attention_tc.cu): bfloat16, 16-key pages, a latent of at most 512.
 bool qb_latent_tc_supports(const QbLatent &a);
 int qb_launch_latent_split_tc(qb_ctx *ctx, const QbLatent &a, uint32_t n_splits);
+// ... and in fp32 arithmetic, for every shape and both types (latent_attention.cu).
+int qb_launch_latent_split_simt(qb_ctx *ctx, const QbLatent &a, uint32_t n_splits);
 // Spans per sequence that fill the GPU once with ns sequences in the launch.
 uint32_t qb_latent_max_splits(const QbLatent &a, uint32_t ns, uint32_t sms);
 // Floats of part_acc for up to rows_cap prompt rows / n_seqs decode rows.
 size_t qb_latent_part_floats(const QbLatent &a, uint32_t rows_cap, uint32_t n_seqs, uint32_t sms);
 int qb_launch_latent(qb_ctx *ctx, const QbLatent &a);
+
+// ---- attention whose values are its keys (shared_kv_attention.cu) --------------------------------------------------------
+// Grouped-query attention with values that are the key projections themselves.  Per head, queries and keys are divided by
+// their root mean square, weighted and rotated; the softmax has a sink of score 0 without a value; each head's output has
+// a gate.  The cache keeps one vector per token and key/value head, and attention runs over it like absorbed latent attention:
+//     cached [k | rot(w k)]    query [0 .. 0 | w_k q_pass | rot(q)]    score = scale / rms(k) * (query . cached)
+// (the dimensions that a rotation passes need the projection only, the rotated ones are kept a second time).
+struct QbSharedKv {
+    QbLatent at;                              // rank = head size, rot_dim = rot.dims, groups = key/value heads, key_scale, buffers
+    const float *proj = nullptr;              // [S][rows][stride]: q (H*dim) | k (groups*dim) | g (H)
+    uint32_t S = 1, stride = 0;
+    const float *q_norm = nullptr, *k_norm = nullptr;      // [dim]
+    float *key_scale = nullptr;               // [slots][groups]
+};
+uint32_t qb_shared_kv_max_splits(const QbLatent &a, uint32_t ns, uint32_t R, uint32_t sms);
+size_t qb_shared_kv_part_floats(const QbLatent &a, uint32_t rows_cap, uint32_t n_seqs, uint32_t sms);
+int qb_launch_shared_kv(qb_ctx *ctx, const QbSharedKv &a);

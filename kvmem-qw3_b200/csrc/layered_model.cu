@@ -1,8 +1,9 @@
 // Layered models: configuration, weights, per-batch buffers and the forward pass (family "layered" of the executor).
 //
 // A config.json lists the layers -- a mixer with its sizes and an optional dense feed-forward -- and an optional span of
-// layers that runs several times with the same weights.  A "run" is one execution of a layer; every run has a cache or
-// state of its own.  Architectures are rows of the loader table in engine.cu, mixers rows of MIXERS below.
+// layers that runs several times with the same weights; a layer may also name an earlier or later one whose weights it uses.
+// A "run" is one execution of a layer's weights; every run has a cache or state of its own.  Architectures are rows of the
+// loader table in engine.cu and of DESIGNS below (what a design fixes for all its models), mixers rows of MIXERS.
 #include "engine.h"
 #include "json_reader.h"
 #include "layered.h"
@@ -13,32 +14,48 @@
 #include <string>
 
 // ---- description ------------------------------------------------------------------------------------------------------------
-enum class MixerKind { Retention, Latent };
+enum class MixerKind { Retention, Lightning, Mlstm, Latent, SharedKv };
+inline bool is_recurrent(MixerKind k) { return k == MixerKind::Retention || k == MixerKind::Lightning || k == MixerKind::Mlstm; }
 struct RotarySpec {
     uint32_t dims = 0;
     double base = 1.0;
-    bool scaled = false;
+    bool stretched = false, blended = false;     // every pair turns slower by `factor` / a blend by pair (original, fast, slow)
     double factor = 1.0, original = 1.0, fast = 1.0, slow = 1.0;
 };
 struct MixerSpec {
     MixerKind kind = MixerKind::Retention;
-    uint32_t heads = 0, dim = 0, vdim = 0, rot_dim = 0, kv_rank = 0;
-    double scale = 1.0;
+    uint32_t heads = 0, dim = 0, vdim = 0, rot_dim = 0, kv_rank = 0, kv_heads = 0;
+    double scale = 1.0, gate_cap = 1.0;
     std::vector<double> decay;
     RotarySpec rot;
 };
-struct LayerSpec { MixerSpec mixer; uint32_t ff = 0; };             // ff 0: no feed-forward
+struct LayerSpec { MixerSpec mixer; uint32_t ff = 0; int weights_of = -1; };   // ff 0: no feed-forward; weights_of -1: its own
+// What a design fixes for all its models.
+struct Design {
+    const char *architecture;
+    bool center;              // layer norms without bias, else RMS norms
+    bool post_norm;           // a norm on each sublayer's output (times a layer scale), none on its input
+    bool embed_norm;          // the embedding is normalised, else multiplied by embedding.scale
+};
+const Design DESIGNS[] = {
+    {"Kezilix", false, false, true},
+    {"Figonex", true, true, false},
+};
 struct LayeredSpec {
     std::string architecture;
+    const Design *design = nullptr;
+    double embed_scale = 1.0;
     uint32_t vocab = 0, width = 0, loop_start = 0, loop_stop = 0, loop_times = 0;     // loop_times 0: no loop
     double eps = 0.0;
     std::vector<LayerSpec> layers;
 };
-struct LayerRun { uint32_t layer; int pass; };                       // pass: -1 outside the loop
+struct LayerRun { uint32_t layer; int pass; bool opens; };           // pass: -1 outside the loop; opens: first of a pass
 
 struct LayeredLayer {
     QbDense w_in, w_out, w_ukv, w_gate_up, w_down;
-    const float *norm1 = nullptr, *norm2 = nullptr, *lat_norm = nullptr, *sink = nullptr, *powers = nullptr;
+    const float *norm1 = nullptr, *norm2 = nullptr;       // gains (post norm: times the layer scale)
+    const float *lat_norm = nullptr, *sink = nullptr, *powers = nullptr, *mix_norm = nullptr, *i_bias = nullptr, *f_bias = nullptr, *q_norm = nullptr,
+                *k_norm = nullptr;
     QbRotary rot;
 };
 struct QbLayered {
@@ -51,8 +68,10 @@ struct QbLayered {
     const float *embed_norm = nullptr, *final_norm = nullptr, *loop_step = nullptr;
 };
 struct QbLayeredBatch {
-    std::vector<void *> cache;                 // per run: the latent cache of a latent-attention run
-    std::vector<float *> state;                // per run: the state of a retention run
+    std::vector<void *> cache;                 // per run: the paged cache of an attention run
+    std::vector<float *> key_scale;            // ... and its factors per key (attention whose values are its keys)
+    std::vector<float *> state;                // per run: the state of a recurrent run
+    float *row_aux = nullptr;                  // per row and head of a recurrent layer: sums of squares / normalisers
     QbActBuf x, mix, ff, lat;                  // normalised rows, mixer output, feed-forward hidden rows, gathered latents
     float *parts = nullptr, *emb = nullptr, *part_acc = nullptr, *part_ml = nullptr;
     void *q = nullptr, *qa = nullptr;
@@ -90,8 +109,10 @@ int parse_rotary(const Value &mixer, RotarySpec &r) {
     QB_REQUIRE(r.dims % 2 == 0, "config.json: rot.dims must be even");
     const Value *s = v->get("scaling");
     if (s && !s->is_null()) {
-        r.scaled = true;
         QB_TRY(need_num(*s, "factor", r.factor));
+        r.blended = s->get("original") || s->get("fast") || s->get("slow");
+        r.stretched = !r.blended;
+        if (r.stretched) return QB_OK;
         QB_TRY(need_num(*s, "original", r.original));
         QB_TRY(need_num(*s, "fast", r.fast));
         QB_TRY(need_num(*s, "slow", r.slow));
@@ -99,11 +120,15 @@ int parse_rotary(const Value &mixer, RotarySpec &r) {
     return QB_OK;
 }
 
-int parse_retention(const Value &v, MixerSpec &m) {
-    m.kind = MixerKind::Retention;
+int parse_decay(const Value &v, MixerSpec &m) {
     const Value *d = v.get("decay");
     QB_REQUIRE(d && d->items.size() == m.heads, "config.json: decay must list one number per head");
     for (const Value &x : d->items) m.decay.push_back(x.num);
+    return QB_OK;
+}
+int parse_retention(const Value &v, MixerSpec &m) {
+    m.kind = MixerKind::Retention;
+    QB_TRY(parse_decay(v, m));
     QB_REQUIRE(m.rot.dims <= m.dim, "config.json: rot.dims exceeds the head");
     return QB_OK;
 }
@@ -115,7 +140,29 @@ int parse_latent(const Value &v, MixerSpec &m) {
     QB_REQUIRE(m.rot.dims <= m.rot_dim, "config.json: rot.dims exceeds rot_dim");
     return QB_OK;
 }
+int parse_lightning(const Value &v, MixerSpec &m) {
+    m.kind = MixerKind::Lightning;
+    return parse_decay(v, m);
+}
+int parse_mlstm(const Value &v, MixerSpec &m) {
+    m.kind = MixerKind::Mlstm;
+    QB_TRY(need_num(v, "gate_cap", m.gate_cap));
+    QB_REQUIRE(m.gate_cap > 0, "config.json: gate_cap must be positive");
+    return QB_OK;
+}
+int parse_shared_kv(const Value &v, MixerSpec &m) {
+    m.kind = MixerKind::SharedKv;
+    QB_TRY(need_u32(v, "kv_heads", m.kv_heads));
+    QB_TRY(need_num(v, "scale", m.scale));
+    QB_REQUIRE(m.heads % m.kv_heads == 0, "config.json: heads must be a multiple of kv_heads");
+    QB_REQUIRE(m.vdim == m.dim, "config.json: the values are the keys, vdim must equal dim");
+    QB_REQUIRE(m.rot.dims <= m.dim, "config.json: rot.dims exceeds the head");
+    return QB_OK;
+}
 const struct { const char *type; int (*parse)(const Value &, MixerSpec &); } MIXERS[] = {
+    {"lightning", parse_lightning},
+    {"mlstm", parse_mlstm},
+    {"attention", parse_shared_kv},
     {"retention", parse_retention},
     {"latent_attention", parse_latent},
 };
@@ -124,6 +171,14 @@ int parse_spec(const std::string &text, LayeredSpec &s) {
     Value root;
     if (!qbjson::Parser(text.data(), text.size()).parse(root) || root.kind != Value::Object) return bad("not a JSON object");
     if (const Value *a = root.get("architecture")) s.architecture = a->s;
+    for (const Design &d : DESIGNS)
+        if (s.architecture == d.architecture) s.design = &d;
+    if (!s.design) return qb_fail(QB_ERR_UNSUPPORTED, "config.json: architecture '%s' is not known", s.architecture.c_str());
+    if (!s.design->embed_norm) {
+        const Value *e = root.get("embedding");
+        if (!e) return bad("embedding is missing");
+        QB_TRY(need_num(*e, "scale", s.embed_scale));
+    }
     QB_TRY(need_u32(root, "vocab", s.vocab));
     QB_TRY(need_u32(root, "width", s.width));
     const Value *norm = root.get("norm");
@@ -148,7 +203,23 @@ int parse_spec(const std::string &text, LayeredSpec &s) {
             if (kind && kind->s != "dense") return qb_fail(QB_ERR_UNSUPPORTED, "config.json: feed-forward %s is not known", kind->s.c_str());
             QB_TRY(need_u32(*mlp, "ff", L.ff));
         }
+        const Value *of = l.get("weights_of");
+        if (of && !of->is_null()) {
+            if (of->kind != Value::Number || of->num < 0 || of->num >= (double)layers->items.size() || of->num != std::floor(of->num))
+                return bad("weights_of must name a layer");
+            L.weights_of = (int)of->num;
+        }
         s.layers.push_back(std::move(L));
+    }
+    // a chain of weights_of ends at a layer with weights of its own, of the same shape
+    for (uint32_t i = 0; i < s.layers.size(); ++i) {
+        uint32_t j = i, hops = 0;
+        for (; s.layers[j].weights_of >= 0 && hops <= s.layers.size(); ++hops) j = (uint32_t)s.layers[j].weights_of;
+        if (hops > s.layers.size()) return bad("weights_of goes in a circle");
+        const LayerSpec &a = s.layers[i], &b = s.layers[j];
+        if (a.mixer.kind != b.mixer.kind || a.mixer.heads != b.mixer.heads || a.mixer.dim != b.mixer.dim || a.mixer.vdim != b.mixer.vdim || a.ff != b.ff ||
+            a.mixer.kv_heads != b.mixer.kv_heads)
+            return bad("a layer with weights_of must equal the layer it names");
     }
     const Value *loop = root.get("loop");
     if (loop && !loop->is_null()) {
@@ -164,22 +235,24 @@ int parse_spec(const std::string &text, LayeredSpec &s) {
 }
 
 std::vector<LayerRun> list_runs(const LayeredSpec &s) {
-    std::vector<LayerRun> r;
+    std::vector<LayerRun> r;                 // (.layer: the one whose weights run)
     const uint32_t n = (uint32_t)s.layers.size(), a = s.loop_times ? s.loop_start : n, b = s.loop_times ? s.loop_stop : n;
-    for (uint32_t i = 0; i < a; ++i) r.push_back({i, -1});
+    for (uint32_t i = 0; i < a; ++i) r.push_back({i, -1, false});
     for (uint32_t t = 0; t < s.loop_times; ++t)
-        for (uint32_t i = a; i < b; ++i) r.push_back({i, (int)t});
-    for (uint32_t i = b; i < n; ++i) r.push_back({i, -1});
+        for (uint32_t i = a; i < b; ++i) r.push_back({i, (int)t, i == a});
+    for (uint32_t i = b; i < n; ++i) r.push_back({i, -1, false});
+    for (LayerRun &run : r)
+        while (s.layers[run.layer].weights_of >= 0) run.layer = (uint32_t)s.layers[run.layer].weights_of;
     return r;
 }
 
-// Frequencies and amplitude of a rotation.  Scaled: pair i turns at its own frequency where a dimension makes more than
+// Frequencies and amplitude of a rotation.  Stretched: every pair turns at 1 / factor.  Blended: pair i turns at its own frequency where a dimension makes more than
 // `fast` turns over the original context, at 1 / factor of it below `slow` turns, and at a blend in between.
 void rotary_freqs(const RotarySpec &r, std::vector<float> &freq, float &amp) {
     freq.assign(std::max(1u, r.dims / 2), 0.0f);
     amp = 1.0f;
     double lo = 0, hi = 0;
-    if (r.scaled) {
+    if (r.blended) {
         auto at = [&](double turns) { return r.dims * std::log(r.original / (2.0 * M_PI * turns)) / (2.0 * std::log(r.base)); };
         lo = std::max(std::floor(at(r.fast)), 0.0);
         hi = std::min(std::ceil(at(r.slow)), (double)r.dims - 1.0);
@@ -187,7 +260,8 @@ void rotary_freqs(const RotarySpec &r, std::vector<float> &freq, float &amp) {
     }
     for (uint32_t i = 0; i < r.dims / 2; ++i) {
         double f = std::pow(r.base, -2.0 * i / r.dims);
-        if (r.scaled) {
+        if (r.stretched) f /= r.factor;
+        if (r.blended) {
             const double ramp = std::min(std::max(((double)i - lo) / std::max(hi - lo, 0.001), 0.0), 1.0);
             f = f / r.factor * ramp + f * (1.0 - ramp);
         }
@@ -224,21 +298,39 @@ int put_matrix(qb_ctx *ctx, Source &src, const std::string &name, QbDense *w, co
     QB_TRY(find_tensor(src, name, {rows.n, w->cols}, &t));
     return qb_dense_upload(ctx, w, rows, (const uint16_t *)t->data);
 }
-// fp32 copy of a vector (or of a small [a][b] table) on the device, owned by the model.
-int put_f32(qb_ctx *ctx, Source &src, qb_model *m, const std::string &name, std::initializer_list<uint64_t> shape, float dflt, const float **out) {
+// A vector (or a small [a][b] table) widened to fp32.
+int read_f32(Source &src, const std::string &name, std::initializer_list<uint64_t> shape, float dflt, std::vector<float> &v) {
     size_t n = 1;
     for (uint64_t d : shape) n *= d;
-    std::vector<float> v(n, dflt);
-    if (src.file) {
-        const qbst::Tensor *t = nullptr;
-        QB_TRY(find_tensor(src, name, shape, &t));
-        for (size_t i = 0; i < n; ++i) { uint16_t raw; memcpy(&raw, t->data + 2 * i, 2); v[i] = bf16_to_f32(raw); }
-    }
+    v.assign(n, dflt);
+    if (!src.file) return QB_OK;
+    const qbst::Tensor *t = nullptr;
+    QB_TRY(find_tensor(src, name, shape, &t));
+    for (size_t i = 0; i < n; ++i) { uint16_t raw; memcpy(&raw, t->data + 2 * i, 2); v[i] = bf16_to_f32(raw); }
+    return QB_OK;
+}
+// fp32 numbers on the device, owned by the model.
+int keep_f32(qb_ctx *ctx, qb_model *m, const std::vector<float> &v, const float **out) {
     float *dev = nullptr;
     QB_TRY(qb_upload_f32(ctx, v, &dev));
     m->owned_f32.push_back(dev);
     *out = dev;
     return QB_OK;
+}
+int put_f32(qb_ctx *ctx, Source &src, qb_model *m, const std::string &name, std::initializer_list<uint64_t> shape, float dflt, const float **out) {
+    std::vector<float> v;
+    QB_TRY(read_f32(src, name, shape, dflt, v));
+    return keep_f32(ctx, m, v, out);
+}
+// Gain of a sublayer's norm, times the layer scale where the design has one (both bfloat16: the product is exact in fp32).
+int put_gain(qb_ctx *ctx, Source &src, qb_model *m, const std::string &norm, const std::string &scale, uint32_t D, const float **out) {
+    std::vector<float> v, l;
+    QB_TRY(read_f32(src, norm, {D}, 1.0f, v));
+    if (m->layered->spec.design->post_norm) {
+        QB_TRY(read_f32(src, scale, {D}, 0.5f, l));
+        for (uint32_t i = 0; i < D; ++i) v[i] *= l[i];
+    }
+    return keep_f32(ctx, m, v, out);
 }
 QbDenseRows rows_at(uint32_t row0, uint32_t n) {
     QbDenseRows r;
@@ -251,11 +343,31 @@ QbDenseRows rows_grouped(uint32_t row0, uint32_t n, uint32_t group, uint32_t str
     return r;
 }
 
-// The shape of a latent-attention layer as its kernels take it (no buffers).
+// The shape of an attention layer as its kernels take it (no buffers).
 QbLatent latent_shape(const MixerSpec &m, bool f32) {
     QbLatent a;
     a.H = m.heads; a.dim = m.dim; a.rot_dim = m.rot_dim; a.vdim = m.vdim; a.rank = m.kv_rank; a.f32 = f32;
+    if (m.kind == MixerKind::SharedKv) { a.rank = m.dim; a.rot_dim = m.rot.dims; a.groups = m.kv_heads; }
     return a;
+}
+
+// The constants of a recurrent mixer as its kernels take them (no buffers).
+QbRecurrence recurrence_shape(const MixerSpec &m) {
+    QbRecurrence a;
+    a.H = m.heads; a.dim = m.dim; a.vdim = m.vdim;
+    a.gated = m.kind == MixerKind::Mlstm;
+    a.cap = (float)m.gate_cap;
+    a.act = m.kind == MixerKind::Lightning;
+    a.sigmoid_gate = m.kind != MixerKind::Retention;
+    if (m.kind == MixerKind::Retention) a.kscale = 1.0f / sqrtf((float)m.dim);
+    if (m.kind == MixerKind::Mlstm) a.qscale = 1.0f / sqrtf((float)m.dim);
+    a.state_stride = qb_recurrence_state(a.H, a.dim, a.vdim, a.gated);
+    return a;
+}
+// The projection rows of a recurrent mixer: q | k | v | g (| i | f, padded to whole 16-byte rows of fp32 sums).
+uint32_t recurrence_rows(const MixerSpec &m) {
+    const uint32_t n = 2 * m.heads * (m.dim + m.vdim) + (m.kind == MixerKind::Mlstm ? 2 * m.heads : 0);
+    return m.kind == MixerKind::Mlstm ? (n + 3) & ~3u : n;
 }
 
 int build_layer(qb_ctx *ctx, qb_model *m, Source &src, uint32_t i) {
@@ -265,28 +377,38 @@ int build_layer(qb_ctx *ctx, qb_model *m, Source &src, uint32_t i) {
     LayeredLayer &L = Y.layers[i];
     const uint32_t D = Y.spec.width, H = mx.heads;
     const std::string p = "l" + std::to_string(i) + ".", q = p + "mix.", f = p + "mlp.";
-    QB_TRY(put_f32(ctx, src, m, p + "norm1", {D}, 1.0f, &L.norm1));
+    if (S.weights_of >= 0) return QB_OK;
+    QB_TRY(put_gain(ctx, src, m, p + "norm1", p + "ls1", D, &L.norm1));
     std::vector<float> freq;
     rotary_freqs(mx.rot, freq, L.rot.amp);
-    float *fd = nullptr;
-    QB_TRY(qb_upload_f32(ctx, freq, &fd));
-    m->owned_f32.push_back(fd);
-    L.rot.freq = fd;
+    QB_TRY(keep_f32(ctx, m, freq, &L.rot.freq));
     L.rot.dims = mx.rot.dims;
-    if (mx.kind == MixerKind::Retention) {
+    if (is_recurrent(mx.kind)) {
         const uint32_t qk = H * mx.dim, vv = H * mx.vdim;
-        QB_TRY(qb_dense_alloc(ctx, 2 * (qk + vv), D, &L.w_in));
+        QB_TRY(qb_dense_alloc(ctx, recurrence_rows(mx), D, &L.w_in));
         QB_TRY(put_matrix(ctx, src, q + "q", &L.w_in, rows_at(0, qk)));
         QB_TRY(put_matrix(ctx, src, q + "k", &L.w_in, rows_at(qk, qk)));
         QB_TRY(put_matrix(ctx, src, q + "v", &L.w_in, rows_at(2 * qk, vv)));
         QB_TRY(put_matrix(ctx, src, q + "g", &L.w_in, rows_at(2 * qk + vv, vv)));
         std::vector<float> pw;
         for (double d : mx.decay)
-            for (uint32_t n = 0; n <= QB_RET_CHUNK; ++n) pw.push_back((float)std::pow(d, (double)n));
-        float *dev = nullptr;
-        QB_TRY(qb_upload_f32(ctx, pw, &dev));
-        m->owned_f32.push_back(dev);
-        L.powers = dev;
+            for (uint32_t n = 0; n <= QB_REC_CHUNK; ++n) pw.push_back((float)std::pow(d, (double)n));
+        if (!pw.empty()) QB_TRY(keep_f32(ctx, m, pw, &L.powers));
+        if (mx.kind != MixerKind::Retention) QB_TRY(put_f32(ctx, src, m, q + "norm", {vv}, 1.0f, &L.mix_norm));
+        if (mx.kind == MixerKind::Mlstm) {
+            QB_TRY(put_matrix(ctx, src, q + "i", &L.w_in, rows_at(2 * (qk + vv), H)));
+            QB_TRY(put_matrix(ctx, src, q + "f", &L.w_in, rows_at(2 * (qk + vv) + H, H)));
+            QB_TRY(put_f32(ctx, src, m, q + "i.b", {H}, 0.0f, &L.i_bias));
+            QB_TRY(put_f32(ctx, src, m, q + "f.b", {H}, 3.0f, &L.f_bias));
+        }
+    } else if (mx.kind == MixerKind::SharedKv) {
+        const uint32_t qd = H * mx.dim, kd = mx.kv_heads * mx.dim;
+        QB_TRY(qb_dense_alloc(ctx, qd + kd + H, D, &L.w_in));
+        QB_TRY(put_matrix(ctx, src, q + "q", &L.w_in, rows_at(0, qd)));
+        QB_TRY(put_matrix(ctx, src, q + "k", &L.w_in, rows_at(qd, kd)));
+        QB_TRY(put_matrix(ctx, src, q + "g", &L.w_in, rows_at(qd + kd, H)));
+        QB_TRY(put_f32(ctx, src, m, q + "q.norm", {mx.dim}, 1.0f, &L.q_norm));
+        QB_TRY(put_f32(ctx, src, m, q + "k.norm", {mx.dim}, 1.0f, &L.k_norm));
     } else {
         L.rot.interleaved = true;
         const QbLatent a = latent_shape(mx, Y.f32);
@@ -305,7 +427,7 @@ int build_layer(qb_ctx *ctx, qb_model *m, Source &src, uint32_t i) {
     QB_TRY(put_matrix(ctx, src, q + "o", &L.w_out, rows_at(0, D)));
     m->weight_bytes += L.w_in.bytes() + L.w_out.bytes() + L.w_ukv.bytes();
     if (S.ff) {
-        QB_TRY(put_f32(ctx, src, m, p + "norm2", {D}, 1.0f, &L.norm2));
+        QB_TRY(put_gain(ctx, src, m, p + "norm2", p + "ls2", D, &L.norm2));
         QB_TRY(qb_dense_alloc(ctx, (S.ff + 15) / 16 * 32, D, &L.w_gate_up));
         QB_TRY(put_matrix(ctx, src, f + "gate", &L.w_gate_up, rows_grouped(0, S.ff, 16, 32)));
         QB_TRY(put_matrix(ctx, src, f + "up", &L.w_gate_up, rows_grouped(16, S.ff, 16, 32)));
@@ -335,7 +457,7 @@ int build_model(qb_ctx *ctx, qb_model *m, Source &src) {
         synth_embed_kernel<<<(unsigned)(((uint64_t)V * D + 255) / 256), 256, 0, ctx->stream>>>(Y.embed, (uint64_t)V * D, src.seed);
         QB_LAUNCHED(ctx, "synth_embed_kernel");
     }
-    QB_TRY(put_f32(ctx, src, m, "embed.norm", {D}, 1.0f, &Y.embed_norm));
+    if (s.design->embed_norm) QB_TRY(put_f32(ctx, src, m, "embed.norm", {D}, 1.0f, &Y.embed_norm));
     if (s.loop_times) QB_TRY(put_f32(ctx, src, m, "loop.step", {s.loop_times, D}, 0.1f, &Y.loop_step));
     QB_TRY(put_f32(ctx, src, m, "final.norm", {D}, 1.0f, &Y.final_norm));
     QB_TRY(qb_dense_alloc(ctx, V, D, &Y.head));
@@ -371,15 +493,25 @@ int layered_batch_alloc(qb_ctx *ctx, qb_batch *b, size_t slots) {
         parts = std::max(parts, (size_t)rows * w.rows);
     };
     uint32_t mix = 1, ff = 1, max_keys = b->pages_per_seq * b->page_size;
-    size_t q = 0, qa = 0, acc = 0, ml = 0, kr = 0, kv = 0, lat_ld = 0;
+    size_t q = 0, qa = 0, acc = 0, ml = 0, kr = 0, kv = 0, lat_ld = 0, aux = 0;
     for (uint32_t i = 0; i < Y.layers.size(); ++i) {
         const LayeredLayer &L = Y.layers[i];
         const LayerSpec &S = Y.spec.layers[i];
         consider(L.w_in); consider(L.w_out); consider(L.w_gate_up); consider(L.w_down);
         mix = std::max(mix, S.mixer.heads * S.mixer.vdim);
         ff = std::max(ff, S.ff);
-        if (S.mixer.kind != MixerKind::Latent) continue;
+        if (is_recurrent(S.mixer.kind)) {
+            if (S.mixer.kind != MixerKind::Retention) aux = std::max(aux, (size_t)rows * S.mixer.heads * 2);
+            continue;
+        }
         const QbLatent a = latent_shape(S.mixer, f32);
+        if (S.mixer.kind == MixerKind::SharedKv) {
+            const size_t pf = qb_shared_kv_part_floats(a, rows, b->n_seqs, sms);
+            qa = std::max(qa, (size_t)rows * a.H * a.pitch());
+            acc = std::max(acc, pf);
+            ml = std::max(ml, pf / a.rank * 2);
+            continue;
+        }
         q = std::max(q, (size_t)rows * a.H * (a.dimp() + a.rotp()));
         qa = std::max(qa, (size_t)rows * a.H * a.pitch());
         const size_t pf = qb_latent_part_floats(a, rows, b->n_seqs, sms);
@@ -396,8 +528,9 @@ int layered_batch_alloc(qb_ctx *ctx, qb_batch *b, size_t slots) {
     QB_TRY(qb_act_alloc(ctx, &B->ff, rows, ff, f32));
     QB_CUDA(cudaMalloc(&B->parts, parts * sizeof(float)));
     QB_CUDA(cudaMalloc(&B->emb, (size_t)rows * D * sizeof(float)));
-    if (q) {
-        QB_CUDA(cudaMalloc(&B->q, q * es));
+    if (aux) QB_CUDA(cudaMalloc(&B->row_aux, aux * sizeof(float)));
+    if (q) QB_CUDA(cudaMalloc(&B->q, q * es));
+    if (qa) {
         QB_CUDA(cudaMalloc(&B->qa, qa * es));
         QB_CUDA(cudaMalloc(&B->part_acc, acc * sizeof(float)));
         QB_CUDA(cudaMalloc(&B->part_ml, ml * sizeof(float)));
@@ -408,16 +541,22 @@ int layered_batch_alloc(qb_ctx *ctx, qb_batch *b, size_t slots) {
         QB_CUDA(cudaMalloc(&B->kv, kv * 2));
     }
     B->cache.assign(Y.runs.size(), nullptr);
+    B->key_scale.assign(Y.runs.size(), nullptr);
     B->state.assign(Y.runs.size(), nullptr);
     for (size_t r = 0; r < Y.runs.size(); ++r) {
         const MixerSpec &mx = Y.spec.layers[Y.runs[r].layer].mixer;
-        if (mx.kind == MixerKind::Latent) {
-            const size_t bytes = slots * latent_shape(mx, f32).pitch() * es;
+        if (!is_recurrent(mx.kind)) {
+            const QbLatent a = latent_shape(mx, f32);
+            const size_t bytes = slots * a.groups * a.pitch() * es;
             QB_CUDA(cudaMalloc(&B->cache[r], bytes));
             QB_CUDA(cudaMemsetAsync(B->cache[r], 0, bytes, ctx->stream));
+            if (mx.kind == MixerKind::SharedKv) {
+                QB_CUDA(cudaMalloc(&B->key_scale[r], slots * a.groups * sizeof(float)));
+                QB_CUDA(cudaMemsetAsync(B->key_scale[r], 0, slots * a.groups * sizeof(float), ctx->stream));
+            }
         } else {
             StateBlock sb;
-            sb.per_seq = sb.head = (size_t)mx.heads * mx.dim * mx.vdim;
+            sb.per_seq = sb.head = recurrence_shape(mx).state_stride;
             QB_CUDA(cudaMalloc(&B->state[r], b->n_seqs * sb.per_seq * sizeof(float)));
             QB_CUDA(cudaMemsetAsync(B->state[r], 0, b->n_seqs * sb.per_seq * sizeof(float), ctx->stream));
             sb.buf[0] = B->state[r];
@@ -432,7 +571,8 @@ void layered_batch_free(qb_batch *b) {
     if (!B) return;
     for (void *p : B->cache) if (p) cudaFree(p);
     for (float *p : B->state) if (p) cudaFree(p);
-    void *ptrs[] = {B->x.p, B->mix.p, B->ff.p, B->lat.p, B->parts, B->emb, B->part_acc, B->part_ml, B->q, B->qa, B->kr, B->kv, B->trace};
+    for (float *p : B->key_scale) if (p) cudaFree(p);
+    void *ptrs[] = {B->x.p, B->mix.p, B->ff.p, B->lat.p, B->parts, B->emb, B->part_acc, B->part_ml, B->q, B->qa, B->kr, B->kv, B->trace, B->row_aux};
     for (void *p : ptrs) if (p) cudaFree(p);
     delete B;
     b->layered = nullptr;
@@ -445,19 +585,51 @@ int product(qb_ctx *ctx, QbLayeredBatch *B, const QbDense &w, const QbActBuf &x,
     return qb_dense_gemm(ctx, w, x, rows, B->parts, *S);
 }
 
-int retention_block(qb_ctx *ctx, qb_batch *b, uint32_t run, const RowSet &rs, uint32_t *S) {
+int recurrent_block(qb_ctx *ctx, qb_batch *b, uint32_t run, const RowSet &rs, uint32_t *S) {
     const QbLayered &Y = *b->m->layered;
     QbLayeredBatch *B = b->layered;
     const LayeredLayer &L = Y.layers[Y.runs[run].layer];
     const MixerSpec &mx = Y.spec.layers[Y.runs[run].layer].mixer;
-    QbRetention a;
+    QbRecurrence a = recurrence_shape(mx);
     QB_TRY(product(ctx, B, L.w_in, B->x, rs.rows(), &a.S));
     a.proj = B->parts; a.stride = L.w_in.rows;
-    a.ns = rs.ns; a.R = rs.R; a.H = mx.heads; a.dim = mx.dim; a.vdim = mx.vdim; a.eps = (float)Y.spec.eps;
+    a.ns = rs.ns; a.R = rs.R; a.eps = (float)Y.spec.eps;
     a.rot = L.rot; a.powers = L.powers; a.seq_pos = rs.seq_pos;
-    a.state = B->state[run] + (size_t)rs.seq0 * mx.heads * mx.dim * mx.vdim;
+    a.norm_w = L.mix_norm; a.i_bias = L.i_bias; a.f_bias = L.f_bias;
+    if (mx.kind == MixerKind::Lightning) a.row_ss = B->row_aux;
+    if (a.gated) a.row_aux = B->row_aux;
+    a.state = B->state[run] + (size_t)rs.seq0 * a.state_stride;
     a.out = B->mix;
-    QB_TRY(qb_launch_retention(ctx, a));
+    QB_TRY(qb_launch_recurrence(ctx, a));
+    return product(ctx, B, L.w_out, B->mix, rs.rows(), S);
+}
+
+// Fields that the attention mixers share: rows, positions, pages, cache, span buffers.
+void attention_common(const qb_batch *b, uint32_t run, const RowSet &rs, const LayeredLayer &L, const MixerSpec &mx, QbLatent &a) {
+    QbLayeredBatch *B = b->layered;
+    a.ns = rs.ns; a.R = rs.R; a.eps = (float)b->m->layered->spec.eps; a.scale = (float)mx.scale;
+    a.rot = L.rot;
+    a.seq_pos = rs.seq_pos; a.max_pos = rs.max_pos; a.ingest = rs.ingest;
+    a.page_table = b->page_table + (size_t)rs.seq0 * b->pages_per_seq; a.pt_stride = b->pages_per_seq; a.page_size = b->page_size;
+    a.cache = B->cache[run];
+    a.slots = b->slots;
+    a.qa = B->qa; a.part_acc = B->part_acc; a.part_ml = B->part_ml;
+    a.out = B->mix;
+}
+
+int shared_kv_block(qb_ctx *ctx, qb_batch *b, uint32_t run, const RowSet &rs, uint32_t *S) {
+    const QbLayered &Y = *b->m->layered;
+    QbLayeredBatch *B = b->layered;
+    const LayeredLayer &L = Y.layers[Y.runs[run].layer];
+    const MixerSpec &mx = Y.spec.layers[Y.runs[run].layer].mixer;
+    QbSharedKv a;
+    a.at = latent_shape(mx, Y.f32);
+    QB_TRY(product(ctx, B, L.w_in, B->x, rs.rows(), &a.S));
+    attention_common(b, run, rs, L, mx, a.at);
+    a.at.max_splits = qb_shared_kv_max_splits(a.at, rs.ns, rs.R, (uint32_t)ctx->sm_count);
+    a.proj = B->parts; a.stride = L.w_in.rows;
+    a.q_norm = L.q_norm; a.k_norm = L.k_norm; a.key_scale = B->key_scale[run];
+    QB_TRY(qb_launch_shared_kv(ctx, a));
     return product(ctx, B, L.w_out, B->mix, rs.rows(), S);
 }
 
@@ -469,15 +641,10 @@ int latent_block(qb_ctx *ctx, qb_batch *b, uint32_t run, const RowSet &rs, uint3
     QbLatent a = latent_shape(mx, Y.f32);
     QB_TRY(product(ctx, B, L.w_in, B->x, rs.rows(), &a.S));
     a.proj = B->parts; a.stride = L.w_in.rows;
-    a.ns = rs.ns; a.R = rs.R; a.eps = (float)Y.spec.eps; a.scale = (float)mx.scale;
-    a.rot = L.rot; a.norm_w = L.lat_norm; a.sink = L.sink; a.ukv = &L.w_ukv;
-    a.seq_pos = rs.seq_pos; a.max_pos = rs.max_pos; a.ingest = rs.ingest;
-    a.page_table = b->page_table + (size_t)rs.seq0 * b->pages_per_seq; a.pt_stride = b->pages_per_seq; a.page_size = b->page_size;
-    a.cache = B->cache[run];
-    a.slots = b->slots;
+    attention_common(b, run, rs, L, mx, a);
+    a.norm_w = L.lat_norm; a.sink = L.sink; a.ukv = &L.w_ukv;
     a.max_splits = qb_latent_max_splits(a, rs.ns, (uint32_t)ctx->sm_count);
-    a.q = B->q; a.qa = B->qa; a.part_acc = B->part_acc; a.part_ml = B->part_ml; a.lat = B->lat; a.kr = B->kr; a.kv = B->kv;
-    a.out = B->mix;
+    a.q = B->q; a.lat = B->lat; a.kr = B->kr; a.kv = B->kv;
     QB_TRY(qb_launch_latent(ctx, a));
     return product(ctx, B, L.w_out, B->mix, rs.rows(), S);
 }
@@ -488,22 +655,27 @@ int layered_forward(qb_ctx *ctx, qb_batch *b, const int32_t *tokens_dev, const R
     const LayeredSpec &s = Y.spec;
     QbLayeredBatch *B = b->layered;
     const uint32_t rows = rs.rows(), D = s.width, n_runs = (uint32_t)Y.runs.size();
-    // The norm launch that opens run r (r = n_runs: the output norm), with what the loop adds in front of a pass.
+    const Design &d = *s.design;
+    auto norm_launch = [&]() {
+        QbLayerNorm n;
+        n.M = rows; n.n = D; n.eps = (float)s.eps; n.center = d.center; n.x = b->hid; n.out = B->x;
+        return n;
+    };
+    // What the norm launch before run r (r = n_runs: the output norm) does for it, with what the loop adds in front of a pass.
     auto open_run = [&](QbLayerNorm &n, uint32_t r) {
-        n.M = rows; n.n = D; n.eps = (float)s.eps; n.x = b->hid; n.out = B->x;
         if (r == n_runs) { n.w = Y.final_norm; return; }
         const LayerRun &run = Y.runs[r];
-        n.w = Y.layers[run.layer].norm1;
-        if (run.pass >= 0 && run.layer == s.loop_start) {
+        n.w = d.post_norm ? nullptr : Y.layers[run.layer].norm1;
+        if (run.opens) {
             if (run.pass > 0) n.emb_add = B->emb;
             n.step = Y.loop_step + (size_t)run.pass * D;
         }
     };
     B->trace_rows = rows;
     {
-        QbLayerNorm n;
+        QbLayerNorm n = norm_launch();
         open_run(n, 0);
-        n.tokens = tokens_dev; n.embed = Y.embed; n.embed_w = Y.embed_norm; n.vocab = s.vocab;
+        n.tokens = tokens_dev; n.embed = Y.embed; n.embed_w = Y.embed_norm; n.embed_scale = (float)s.embed_scale; n.vocab = s.vocab;
         n.emb_store = s.loop_times > 1 ? B->emb : nullptr;
         QB_TRY(qb_launch_layer_norm(ctx, n));
     }
@@ -511,19 +683,23 @@ int layered_forward(qb_ctx *ctx, qb_batch *b, const int32_t *tokens_dev, const R
         const LayeredLayer &L = Y.layers[Y.runs[r].layer];
         const LayerSpec &S = s.layers[Y.runs[r].layer];
         uint32_t seg = 1;
-        if (S.mixer.kind == MixerKind::Retention) QB_TRY(retention_block(ctx, b, r, rs, &seg));
+        if (is_recurrent(S.mixer.kind)) QB_TRY(recurrent_block(ctx, b, r, rs, &seg));
+        else if (S.mixer.kind == MixerKind::SharedKv) QB_TRY(shared_kv_block(ctx, b, r, rs, &seg));
         else QB_TRY(latent_block(ctx, b, r, rs, &seg));
+        QbLayerNorm n = norm_launch();                       // after the mixer
+        if (S.mixer.kind == MixerKind::Lightning) { n.row_ss = B->row_aux; n.ss_n = S.mixer.heads; n.ss_len = S.mixer.heads * S.mixer.vdim; }
+        n.parts = B->parts; n.S = seg;
+        if (d.post_norm) n.post_w = L.norm1;
         if (S.ff) {
-            QbLayerNorm n;
-            n.M = rows; n.n = D; n.eps = (float)s.eps; n.x = b->hid; n.out = B->x;
-            n.parts = B->parts; n.S = seg; n.w = L.norm2;
+            if (!d.post_norm) n.w = L.norm2;
             QB_TRY(qb_launch_layer_norm(ctx, n));
             QB_TRY(qb_dense_gate_up(ctx, L.w_gate_up, B->x, rows, S.ff, B->parts, B->ff));
             QB_TRY(product(ctx, B, L.w_down, B->ff, rows, &seg));
+            n = norm_launch();                               // after the feed-forward
+            n.parts = B->parts; n.S = seg;
+            if (d.post_norm) n.post_w = L.norm2;
         }
-        QbLayerNorm n;
         open_run(n, r + 1);
-        n.parts = B->parts; n.S = seg;
         if (B->trace) n.trace = B->trace + (size_t)r * b->rows_cap * D;
         QB_TRY(qb_launch_layer_norm(ctx, n));
     }
@@ -535,7 +711,7 @@ int layered_head(qb_ctx *ctx, qb_batch *b, const int32_t *row_map, uint32_t rows
     QbLayeredBatch *B = b->layered;
     if (row_map) {
         QbLayerNorm n;
-        n.M = rows; n.n = Y.spec.width; n.eps = (float)Y.spec.eps; n.x = b->hid; n.x_rows = b->rows_cap + b->n_seqs; n.row_map = row_map; n.w = Y.final_norm; n.out = B->x;
+        n.M = rows; n.n = Y.spec.width; n.eps = (float)Y.spec.eps; n.center = Y.spec.design->center; n.x = b->hid; n.x_rows = b->rows_cap + b->n_seqs; n.row_map = row_map; n.w = Y.final_norm; n.out = B->x;
         QB_TRY(qb_launch_layer_norm(ctx, n));
     }
     return qb_dense_gemm(ctx, Y.head, B->x, rows, dst, 1);

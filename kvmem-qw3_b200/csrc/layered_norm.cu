@@ -1,4 +1,5 @@
-// Residual addition, the loop's additions and the RMS norm that follows, in one launch (layered models).
+// The residual stream between two sublayers in one launch (layered models): the sublayer's result -- plain, or normalised and
+// weighted first -- joins the stream, then the loop's additions, then the norm of what follows (or its plain cast).
 #include "layered.h"
 
 namespace {
@@ -33,11 +34,38 @@ template <int V> __device__ __forceinline__ void add(Vec<V> &a, const Vec<V> &b)
 #pragma unroll
     for (int i = 0; i < V; ++i) a.v[i] += b.v[i];
 }
-template <int V> __device__ __forceinline__ float sq(const Vec<V> &a) {
+template <int V> __device__ __forceinline__ float sum(const Vec<V> &a) {
     float s = 0.0f;
 #pragma unroll
-    for (int i = 0; i < V; ++i) s += a.v[i] * a.v[i];
+    for (int i = 0; i < V; ++i) s += a.v[i];
     return s;
+}
+// squares of the deviations from a mean (0: plain squares)
+template <int V> __device__ __forceinline__ float sq(const Vec<V> &a, float mean) {
+    float s = 0.0f;
+#pragma unroll
+    for (int i = 0; i < V; ++i) { const float d = a.v[i] - mean; s += d * d; }
+    return s;
+}
+
+// Mean (0 for an RMS norm) and 1 / root of the mean square of a row whose pieces a block's threads hold.
+struct Moments { float mean, inv; };
+template <int V, int NE>
+__device__ __forceinline__ Moments moments(const Vec<V> (&row)[NE], const QbLayerNorm &a, float *red) {
+    Moments r{0.0f, 1.0f};
+    if (a.center) {
+        float t = 0.0f;
+#pragma unroll
+        for (int k = 0; k < NE; ++k)
+            if ((threadIdx.x + k * LN_THREADS) * V < a.n) t += sum(row[k]);
+        r.mean = qb_block_sum(t, red, LN_THREADS / 32) / (float)a.n;
+    }
+    float ss = 0.0f;
+#pragma unroll
+    for (int k = 0; k < NE; ++k)
+        if ((threadIdx.x + k * LN_THREADS) * V < a.n) ss += sq(row[k], r.mean);
+    r.inv = rsqrtf(qb_block_sum(ss, red, LN_THREADS / 32) / (float)a.n + a.eps);
+    return r;
 }
 
 // One CTA per row; a thread keeps its NE pieces of the row in registers.
@@ -57,29 +85,41 @@ layer_norm_kernel(QbLayerNorm a) {
     if (a.tokens) {
         const uint32_t t = (uint32_t)a.tokens[m];
         const __nv_bfloat16 *e = a.embed + (size_t)(t < a.vocab ? t : 0) * n;
-        float ss = 0.0f;
-#pragma unroll
-        for (int k = 0; k < NE; ++k) {
-            const uint32_t i = (tid + k * LN_THREADS) * V;
-            if (i < n) { row[k] = ld<V>(e + i); ss += sq(row[k]); }
-        }
-        const float inv = rsqrtf(qb_block_sum(ss, red, LN_THREADS / 32) / (float)n + a.eps);
 #pragma unroll
         for (int k = 0; k < NE; ++k) {
             const uint32_t i = (tid + k * LN_THREADS) * V;
             if (i < n) {
-                const Vec<V> w = ld<V>(a.embed_w + i);
+                row[k] = ld<V>(e + i);
 #pragma unroll
-                for (int j = 0; j < V; ++j) row[k].v[j] = row[k].v[j] * inv * w.v[j];
+                for (int j = 0; j < V; ++j) row[k].v[j] *= a.embed_scale;
+            }
+        }
+        if (a.embed_w) {
+            const Moments mo = moments<V, NE>(row, a, red);
+#pragma unroll
+            for (int k = 0; k < NE; ++k) {
+                const uint32_t i = (tid + k * LN_THREADS) * V;
+                if (i < n) {
+                    const Vec<V> w = ld<V>(a.embed_w + i);
+#pragma unroll
+                    for (int j = 0; j < V; ++j) row[k].v[j] = (row[k].v[j] - mo.mean) * mo.inv * w.v[j];
+                }
             }
         }
     } else {
         const size_t ps = (size_t)a.M * n;
+        Vec<V> res[NE];
+        float scale = 1.0f;
+        if (a.row_ss) {                                           // the norm that the mixer left out of its rows
+            float t = 0.0f;
+            for (uint32_t i = 0; i < a.ss_n; ++i) t += a.row_ss[(size_t)m * a.ss_n + i];
+            scale = rsqrtf(t / (float)a.ss_len + a.eps);
+        }
 #pragma unroll
         for (int k = 0; k < NE; ++k) {
             const uint32_t i = (tid + k * LN_THREADS) * V;
             if (i < n) {
-                row[k] = ld<V>(x + i);
+                res[k] = ld<V>(x + i);
                 if (a.S) {
                     const float *p = a.parts + (size_t)m * n + i;
                     Vec<V> sum = ld<V>(p);
@@ -92,12 +132,31 @@ layer_norm_kernel(QbLayerNorm a) {
                         for (uint32_t s = 1; s < 8; ++s)
                             if (s < a.S) add(sum, q[s - 1]);
                     }
-                    add(row[k], sum);
+                    row[k] = sum;
+#pragma unroll
+                    for (int j = 0; j < V; ++j) row[k].v[j] *= scale;
                 }
             }
         }
+        if (a.post_w) {
+            const Moments mo = moments<V, NE>(row, a, red);
+#pragma unroll
+            for (int k = 0; k < NE; ++k) {
+                const uint32_t i = (tid + k * LN_THREADS) * V;
+                if (i < n) {
+                    const Vec<V> w = ld<V>(a.post_w + i);
+#pragma unroll
+                    for (int j = 0; j < V; ++j) row[k].v[j] = (row[k].v[j] - mo.mean) * mo.inv * w.v[j];
+                }
+            }
+        }
+#pragma unroll
+        for (int k = 0; k < NE; ++k) {
+            if ((tid + k * LN_THREADS) * V >= n) continue;
+            if (a.S) add(row[k], res[k]);
+            else row[k] = res[k];
+        }
     }
-    float ss = 0.0f;
 #pragma unroll
     for (int k = 0; k < NE; ++k) {
         const uint32_t i = (tid + k * LN_THREADS) * V;
@@ -108,19 +167,25 @@ layer_norm_kernel(QbLayerNorm a) {
             if (a.emb_add) add(row[k], ld<V>(a.emb_add + at));
             if (a.step) add(row[k], ld<V>(a.step + i));
             if (!a.row_map) st<V>(x + i, row[k]);
-            ss += sq(row[k]);
         }
     }
-    if (!a.w) return;
-    const float inv = rsqrtf(qb_block_sum(ss, red, LN_THREADS / 32) / (float)n + a.eps);
     T *out = (T *)a.out.p + (size_t)m * a.out.ld;
+    if (!a.w) {
+#pragma unroll
+        for (int k = 0; k < NE; ++k) {
+            const uint32_t i = (tid + k * LN_THREADS) * V;
+            if (i < n) st<V>(out + i, row[k]);
+        }
+        return;
+    }
+    const Moments mo = moments<V, NE>(row, a, red);
 #pragma unroll
     for (int k = 0; k < NE; ++k) {
         const uint32_t i = (tid + k * LN_THREADS) * V;
         if (i < n) {
             Vec<V> w = ld<V>(a.w + i);
 #pragma unroll
-            for (int j = 0; j < V; ++j) w.v[j] = row[k].v[j] * inv * w.v[j];
+            for (int j = 0; j < V; ++j) w.v[j] = (row[k].v[j] - mo.mean) * mo.inv * w.v[j];
             st<V>(out + i, w);
         }
     }
@@ -145,7 +210,7 @@ int qb_launch_layer_norm(qb_ctx *ctx, const QbLayerNorm &args) {
     QbLayerNorm a = args;
     a.err_flag = ctx->err_flag_dev;
     QB_REQUIRE(a.M > 0, "layer norm: no rows");
-    QB_REQUIRE(!a.w || (a.M <= a.out.cap && a.n <= a.out.ld), "layer norm: %u rows of %u elements exceed the output buffer", a.M, a.n);
+    QB_REQUIRE(a.out.p && a.M <= a.out.cap && a.n <= a.out.ld, "layer norm: %u rows of %u elements exceed the output buffer", a.M, a.n);
     if (a.n % 4 == 0) return a.out.f32 ? launch<float, 4>(ctx, a) : launch<__nv_bfloat16, 4>(ctx, a);
     return a.out.f32 ? launch<float, 1>(ctx, a) : launch<__nv_bfloat16, 1>(ctx, a);
 }
