@@ -24,6 +24,7 @@ Other workloads, one GPU, for profiling (each prints its own lines):
     --workload timeline  per-launch device timeline of the tensor-core GEMMs of one step
     --workload serve     the continuous-batching loops at the 27B shape, wall clock
     --workload kezilix   prefill and decode of the Kezilix design beside the qwen35 hybrid at equal size, per kernel
+    --workload figonex   the same for the Figonex design, beside Kezilix and qwen35
     --workload tokenizer the byte-level BPE tokenizer on the host (no GPU): MB/s beside the reference's own, where built
 """
 import argparse
@@ -57,7 +58,7 @@ def parse_args():
     ap.add_argument("--steps", type=int, default=40)
     ap.add_argument("--warmup", type=int, default=4)
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
-    ap.add_argument("--workload", default="step", choices=["step", "gemm", "attn", "timeline", "serve", "kezilix", "tokenizer"])
+    ap.add_argument("--workload", default="step", choices=["step", "gemm", "attn", "timeline", "serve", "kezilix", "figonex", "tokenizer"])
     ap.add_argument("--sub", default="all", choices=["all", "none"], help="the short runs of configurations 3, 4, 5 / the TP FFN pair")
     ap.add_argument("--layers", type=int, default=64, help="target layers (64 = the 27B-class shape)")
     ap.add_argument("--prompt", type=int, default=PROMPT_LEN)
@@ -72,7 +73,7 @@ def parse_args():
     ap.add_argument("--impls", default="1,2")
     ap.add_argument("--ctx", default="2048,32768")
     ap.add_argument("--tp", action="store_true", help="--workload gemm: the tensor-parallel FFN pair over the ranks of this launch")
-    ap.add_argument("--sizes", default="2048x6144,4096x12288,5120x17408", help="--workload kezilix: width x feed-forward size, comma list")
+    ap.add_argument("--sizes", default="2048x6144,4096x12288,5120x17408", help="--workload kezilix / figonex: width x feed-forward size, comma list")
     ap.add_argument("--slots", type=int, default=8)
     ap.add_argument("--requests", type=int, default=24)
     return ap.parse_args()
@@ -897,29 +898,35 @@ def family_bounds(family, cfg, rows, keys, ingest):
     per forward; keys: {sequence: context} -> number of keys each decode row attends, or the prompt length (ingest)."""
     hbm, _ = peaks()
     us = lambda nbytes, tflop=0.0, peak=1.0: max(nbytes / hbm * 1e-3, tflop / peak * 1e6)
-    out = {"gemm": 0.0, "recurrent": 0.0, "attention": 0.0, "norm": 0.0}
-    if family == "kezilix":
+    out = {"gemm": 0.0, "recurrent": 0.0, "gated": 0.0, "attention": 0.0, "norm": 0.0}
+    layered = family in ("kezilix", "figonex")
+    if layered:
         D, V, L = cfg["width"], cfg["vocab"], cfg["layers"]
         ff = L[0]["mlp"]["ff"]
     else:
         D, V, ff = cfg.n_embd, cfg.vocab_size, cfg.n_ff
         L = [{"type": "latent_attention" if (i + 1) % 4 == 0 else "retention"} for i in range(cfg.n_layers)]
-    wb, peak = (2.0, bf16_peak()) if family == "kezilix" else (34.0 / 32.0, INT8_PEAK_TOPS)
+    wb, peak = (2.0, bf16_peak()) if layered else (34.0 / 32.0, INT8_PEAK_TOPS)
 
     def gemm(N, Kd, m=None):
         m = m or rows
         out["gemm"] += us(N * Kd * wb + m * Kd * wb + m * N * 4.0, 2.0 * m * N * Kd * 1e-12, peak)
     pairs = float(keys) * (keys + 1) / 2 if ingest else float(rows) * keys
     for l in L:
-        recurrent = l["type"] == "retention"
-        if family == "kezilix":
+        recurrent = l["type"] in ("retention", "lightning", "mlstm")
+        if layered:
             m = l["mixer"]
             H, d, v = m["heads"], m["dim"], m["vdim"]
             if recurrent:
-                gemm(2 * H * (d + v), D)
-                st = 2.0 * H * d * v * 4 * (1 if ingest else rows)
-                fl = rows * H * (2.0 * d * v * 2 + (64 * (d + v) if ingest else 0))
-                out["recurrent"] += us(st + rows * 2.0 * H * (d + v) * 4 + rows * H * v * 2, fl * 1e-12, FP32_PEAK_TFLOPS)
+                gated = l["type"] == "mlstm"
+                gemm(2 * H * (d + v) + 2 * H * gated, D)
+                st = 2.0 * H * d * (v + gated) * 4 * (1 if ingest else rows)
+                fl = rows * H * (2.0 * d * (v + gated) * 2 + (64 * (d + v) if ingest else 0))
+                out["gated" if gated else "recurrent"] += us(st + rows * 2.0 * H * (d + v) * 4 + rows * H * v * 2, fl * 1e-12, FP32_PEAK_TFLOPS)
+            elif l["type"] == "attention":
+                G, c = m["kv_heads"], d + m["rot"]["dims"]                    # numbers per cached vector
+                gemm((H + G) * d + H, D)
+                out["attention"] += us((keys if ingest else rows * keys) * G * (c * 2.0 + 4) + rows * H * d * 4.0, pairs * H * 2 * (c + d) * 1e-12, bf16_peak())
             else:
                 r, k = m["rot_dim"], m["kv_rank"]
                 gemm(H * (d + r) + k + r, D)
@@ -949,7 +956,8 @@ def family_bounds(family, cfg, rows, keys, ingest):
     return out
 
 
-KERNEL_GROUPS = (("gemm", ("gemm",)), ("recurrent", ("retention", "dn_")), ("attention", ("latent", "attn", "qk_norm")), ("norm", ("norm_quant", "layer_norm")))
+KERNEL_GROUPS = (("gemm", ("gemm",)), ("gated", ("gated_recurrence",)), ("recurrent", ("recurrence", "dn_")),
+                 ("attention", ("latent", "shared_kv", "attn", "qk_norm")), ("norm", ("norm_quant", "layer_norm")))
 
 
 def kernel_groups(trace):
@@ -962,9 +970,9 @@ def kernel_groups(trace):
     return out, names
 
 
-def workload_kezilix(args):
-    """Prefill and decode throughput of the Kezilix design (bfloat16) and of the qwen35 hybrid (Q8_0) at equal width,
-    feed-forward size and depth (seeded random weights), with the time of every kernel group beside its bound: weights and
+def workload_layered(args):
+    """Prefill and decode throughput of a layered design (bfloat16) and of the qwen35 hybrid (Q8_0) at equal width,
+    feed-forward size and depth (seeded random weights); of Figonex beside Kezilix as well; with the time of every kernel group beside its bound: weights and
     caches exceed L2, 3 warm-up iterations, CUDA events.  The per-kernel times come from a pass with an event after every
     launch (no overlap between launches, about 2 us each)."""
     pkg = entry.load_package()
@@ -985,9 +993,9 @@ def workload_kezilix(args):
 
     for size in args.sizes.split(","):
         width, ff = map(int, size.split("x"))
-        for family in ("kezilix", "qwen35"):
-            if family == "kezilix":
-                cfg = pkg.configs.kezilix_bench(width, ff)
+        for family in (("kezilix", "qwen35") if args.workload == "kezilix" else ("figonex", "kezilix", "qwen35")):
+            if family != "qwen35":
+                cfg = (pkg.configs.kezilix_bench if family == "kezilix" else pkg.configs.figonex_bench)(width, ff)
                 model, vocab = pkg.Model.layered_synth(ctx, cfg, 7), cfg["vocab"]
             else:
                 cfg = pkg.configs.qwen35_bench(width, ff)
@@ -1090,7 +1098,7 @@ def main():
     local_rank = int(os.environ.get("LOCAL_RANK", "0"))
     if args.workload != "step":
         return {"gemm": workload_gemm, "attn": workload_attn, "timeline": workload_timeline, "serve": workload_serve,
-                "kezilix": workload_kezilix, "tokenizer": workload_tokenizer}[args.workload](args)
+                "kezilix": workload_layered, "figonex": workload_layered, "tokenizer": workload_tokenizer}[args.workload](args)
     if args.impl == "reference":
         run_reference(args, rank)
         return

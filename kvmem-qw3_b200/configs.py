@@ -34,6 +34,23 @@ def kezilix_bench(width, ff, n_layers=8, vocab=32768, loop=None):
             "layers": [lat if (i + 1) % 4 == 0 else ret for i in range(n_layers)]}
 
 
+def figonex_bench(width, ff, n_layers=8, vocab=32768, tied=False):
+    """A Figonex model with layers of a real model's size: every fourth layer attention (heads of 128, 32 rotated dimensions,
+    four query heads per key/value head), the others lightning (heads of 128) and mLSTM (128 x 256) by turns, a feed-forward in
+    every layer.  tied: the second half of the layers uses the weights of the first."""
+    H, dense = width // 128, {"kind": "dense", "ff": ff}
+    att = {"type": "attention", "mlp": dense,
+           "mixer": {"heads": H, "kv_heads": H // 4, "dim": 128, "vdim": 128, "scale": 128 ** -0.5,
+                     "rot": {"dims": 32, "base": 1e4, "scaling": {"factor": 4.0}}}}
+    lig = {"type": "lightning", "mlp": dense,
+           "mixer": {"heads": H, "dim": 128, "vdim": 128, "decay": [1.0 - 2.0 ** -(3.0 + 6.0 * i / H) for i in range(H)]}}
+    mls = {"type": "mlstm", "mlp": dense, "mixer": {"heads": width // 256, "dim": 128, "vdim": 256, "gate_cap": 15.0}}
+    layers = [att if i % 4 == 3 else mls if i % 4 == 1 else lig for i in range(n_layers)]
+    if tied:
+        layers = layers[:n_layers // 2] + [dict(l, weights_of=i) for i, l in enumerate(layers[:n_layers // 2])]
+    return {"architecture": "Figonex", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "embedding": {"scale": width ** 0.5}, "layers": layers}
+
+
 def qwen35_bench(width, ff, n_layers=8, vocab=32768):
     """The qwen35 hybrid at the width, feed-forward size, depth and attention interval of kezilix_bench."""
     return ModelConfig(n_layers=n_layers, n_embd=width, n_ff=ff, n_heads=width // 256, n_kv_heads=4 if width % 1024 == 0 else 2, head_dim=256,

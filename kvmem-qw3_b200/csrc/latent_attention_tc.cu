@@ -28,6 +28,7 @@ template <int NQ>
 struct LtcCfg {
     static constexpr int SM_THREADS = NQ * 8;       // softmax threads: 128 lanes x NQ / 16 column groups
     static constexpr int THREADS = 64 + SM_THREADS;
+    static constexpr int CTAS = NQ <= 16 ? 3 : NQ <= 32 ? 2 : 1;      // resident CTAs per SM that the registers allow (small tiles)
     static constexpr uint32_t OST = NQ <= 32 ? 32 : 64;      // column stride of S and of the blocks of O in tensor memory
 };
 struct LtcSmem { uint32_t q, p, misc, total; };
@@ -46,7 +47,7 @@ __host__ __device__ inline uint32_t ltc_tmem_cols(uint32_t NB, uint32_t ost) {
 
 // grid (spans, query groups, sequences)
 template <int NQ>
-__global__ void __launch_bounds__(LtcCfg<NQ>::THREADS, 1)
+__global__ void __launch_bounds__(LtcCfg<NQ>::THREADS, LtcCfg<NQ>::CTAS)
 latent_split_tc_kernel(QbLatent a, const __grid_constant__ CUtensorMap map, uint32_t n_splits, uint32_t NU, uint32_t NB) {
     using C = LtcCfg<NQ>;
     extern __shared__ uint8_t smem_raw[];

@@ -122,6 +122,9 @@ inline size_t qb_recurrence_state(uint32_t H, uint32_t dim, uint32_t vdim, bool 
     return (n + 3) & ~(size_t)3;
 }
 int qb_launch_recurrence(qb_ctx *ctx, const QbRecurrence &a);
+// The blocks of a prompt chunk on the tensor cores (linear_recurrence_mma.cu): bfloat16 models, heads up to 256.
+bool qb_recurrence_mma_supports(const QbRecurrence &a);
+int qb_launch_recurrence_mma(qb_ctx *ctx, const QbRecurrence &a);
 
 // ---- latent attention (latent_attention.cu) ----------------------------------------------------------------------------
 // Keys and values of all heads come from one latent vector per token; the cache holds the latent and one rotated key part

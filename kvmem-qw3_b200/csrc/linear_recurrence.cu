@@ -13,51 +13,25 @@
 //
 // Prompt chunks (recurrence_chunk_kernel): blocks of 64 rows.  With D[i][j] the decay from row j to row i,
 //     O = (Q K^T . D) V + diag(a_i) Q S        S' = keep S + sum_j w_j k_j v_j^T
-// everything in fp32 on the CUDA cores.  Fixed decays: powers from a table made in double precision.  Gated: with b the
+// everything in fp32 on the CUDA cores (float32 models), or on the tensor cores with operands split into two bfloat16 parts
+// (linear_recurrence_mma.cu).  Fixed decays: powers from a table made in double precision.  Gated: with b the
 // running sum of the log forget gates (double precision), m_i = max(m_0 + b_i, max_j (i_j + b_i - b_j)),
 //     D[i][j] = exp(b_i - b_j + i_j - m_i)   a_i = exp(m_0 + b_i - m_i)   w_j = exp(b_n - b_j + i_j - m_n)   keep = a_n
 // and the division by the normaliser waits for the output kernel.
-#include "layered.h"
+#include "linear_recurrence.cuh"
 
 #include <cooperative_groups.h>
 namespace cg = cooperative_groups;
 
 namespace {
+using namespace qbrec;
 
 constexpr int RT = 256;
-constexpr uint32_t C = QB_REC_CHUNK, VCH = QB_REC_SLICE;
 
 // "This CTA runs": arrived at on entry, awaited before the first store into another CTA's shared memory, which must not be
 // touched before that CTA has started.
 __device__ __forceinline__ void cluster_started() { asm volatile("barrier.cluster.arrive.relaxed.aligned;" ::: "memory"); }
 __device__ __forceinline__ void cluster_wait_started() { asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory"); }
-
-__device__ __forceinline__ float act_in(const QbRecurrence &a, float v) { return a.act ? qb_swiglu(v, 1.0f) : v; }
-__device__ __forceinline__ float gate_out(const QbRecurrence &a, float g) { return a.sigmoid_gate ? qb_sigmoid(g) : qb_swiglu(g, 1.0f); }
-// Log gates of head h from the two projections of a row.
-__device__ __forceinline__ float log_input_gate(const QbRecurrence &a, uint32_t h, float z) { return a.cap * tanhf((z + a.i_bias[h]) / a.cap); }
-__device__ __forceinline__ float log_forget_gate(const QbRecurrence &a, uint32_t h, float z) {
-    const float c = a.cap * tanhf((z + a.f_bias[h]) / a.cap);
-    return fminf(c, 0.0f) - log1pf(expf(-fabsf(c)));
-}
-__device__ __forceinline__ float normaliser(float nq, float m) { return fmaxf(fabsf(nq), expf(-m)) + 1e-6f; }
-// A gated sequence state: [H][dim][vdim], then n [H][dim], then m [H][slices] (a copy per slice of a prompt chunk's CTAs).
-__device__ __forceinline__ float *state_of(const QbRecurrence &a, uint32_t s) { return a.state + (size_t)s * a.state_stride; }
-__device__ __forceinline__ float *state_n(const QbRecurrence &a, uint32_t s, uint32_t h) { return state_of(a, s) + (size_t)a.H * a.dim * a.vdim + (size_t)h * a.dim; }
-__device__ __forceinline__ float *state_m(const QbRecurrence &a, uint32_t s, uint32_t h) {
-    return state_of(a, s) + (size_t)a.H * a.dim * (a.vdim + 1) + (size_t)h * qb_recurrence_slices(a.vdim);
-}
-// One token's gates: decay of the state, weight of the new outer product, and the running maximum moved on.
-struct StepGates { float keep, add, m; };
-__device__ __forceinline__ StepGates step_gates(const QbRecurrence &a, uint32_t h, size_t base, size_t ps, float m) {
-    const uint32_t ib = 2 * a.H * (a.dim + a.vdim);
-    const float i = log_input_gate(a, h, qb_sum8(a.proj, base + ib + h, a.S, ps)), f = log_forget_gate(a, h, qb_sum8(a.proj, base + ib + a.H + h, a.S, ps));
-    StepGates g;
-    g.m = fmaxf(f + m, i);
-    g.keep = expf(f + m - g.m);
-    g.add = expf(i - g.m);
-    return g;
-}
 
 template <typename T, bool GATED>
 __global__ void __launch_bounds__(RT)
@@ -332,10 +306,9 @@ recurrence_chunk_kernel(QbRecurrence a, uint32_t dimr) {
     constexpr uint32_t PP = C + 4;
     float *qs = sm, *ks = qs + C * dp, *vs = ks + C * dp, *st = vs + C * VCH, *pm = st + dimr * VCH, *pw = pm + C * PP;
     float *nst = pw + C + 4;                      // gated: n [dimr]
-    // per block: factor of the incoming state per row, weight of a row in the outgoing state; gated: the sums b, the log input
-    // gates and the running maxima
-    __shared__ float rowf[C], colf[C], ig[C], mr[C], keep_s;
-    __shared__ double bs[C];
+    // per block: factor of the incoming state per row (bg.rowf), weight of a row in the outgoing state
+    __shared__ BlockGates bg;
+    __shared__ float colf[C], keep_s;
     const uint32_t tid = threadIdx.x, h = blockIdx.y, s = blockIdx.z, v0 = blockIdx.x * VCH;
     const uint32_t nv = min(VCH, a.vdim - v0);
     float *gst = state_of(a, s) + (size_t)h * a.dim * a.vdim + v0;
@@ -360,58 +333,41 @@ recurrence_chunk_kernel(QbRecurrence a, uint32_t dimr) {
         for (uint32_t i = tid; i < C * dimr; i += RT) {
             const uint32_t r = i / dimr, d = i % dimr;
             const bool in = r < n && d < a.dim;
-            qs[r * dp + d] = in ? act_in(a, rows[(size_t)r * a.stride + h * a.dim + d]) * a.qscale : 0.0f;
-            ks[r * dp + d] = in ? act_in(a, rows[(size_t)r * a.stride + kb + h * a.dim + d]) * a.kscale : 0.0f;
+            qs[r * dp + d] = in ? rows[(size_t)r * a.stride + h * a.dim + d] : 0.0f;
+            ks[r * dp + d] = in ? rows[(size_t)r * a.stride + kb + h * a.dim + d] : 0.0f;
         }
         for (uint32_t i = tid; i < C * VCH; i += RT) {
             const uint32_t r = i / VCH, c = i % VCH;
-            vs[i] = (r < n && c < nv) ? act_in(a, rows[(size_t)r * a.stride + vb + h * a.vdim + v0 + c]) : 0.0f;
+            vs[i] = (r < n && c < nv) ? rows[(size_t)r * a.stride + vb + h * a.vdim + v0 + c] : 0.0f;
+        }
+        if (a.act || a.qscale != 1.0f || a.kscale != 1.0f) {     // (a thread's own elements; silu(0) = 0)
+            for (uint32_t i = tid; i < C * dimr; i += RT) {
+                const uint32_t at = i / dimr * dp + i % dimr;
+                qs[at] = act_in(a, qs[at]) * a.qscale;
+                ks[at] = act_in(a, ks[at]) * a.kscale;
+            }
+            if (a.act) for (uint32_t i = tid; i < C * VCH; i += RT) vs[i] = act_in(a, vs[i]);
         }
         if constexpr (GATED) {
-            if (tid < 32) {                                      // rows 2 lane, 2 lane + 1: a scan of the sums, then of i_j - b_j
+            if (tid < 32) {
                 const uint32_t gi = 2 * a.H * (a.dim + a.vdim) + h;
-                float iv[2];
-                double f[2], b[2], x[2];
+                float zi[2], zf[2];
 #pragma unroll
                 for (int e = 0; e < 2; ++e) {
-                    const uint32_t r = 2 * tid + e;
-                    const float *row = rows + (size_t)min(r, n - 1) * a.stride + gi;
-                    iv[e] = log_input_gate(a, h, row[0]);
-                    f[e] = (double)log_forget_gate(a, h, row[a.H]);
+                    const float *row = rows + (size_t)min(2 * tid + e, n - 1) * a.stride + gi;
+                    zi[e] = row[0];
+                    zf[e] = row[a.H];
                 }
-                double run = f[0] + f[1];
-                for (uint32_t off = 1; off < 32; off <<= 1) {
-                    const double up = __shfl_up_sync(0xffffffffu, run, off);
-                    if (tid >= off) run += up;
-                }
-                b[1] = run;
-                b[0] = run - f[1];
-                x[0] = (double)iv[0] - b[0];
-                x[1] = fmax(x[0], (double)iv[1] - b[1]);
-                double mx = x[1];
-                for (uint32_t off = 1; off < 32; off <<= 1) {
-                    const double up = __shfl_up_sync(0xffffffffu, mx, off);
-                    if (tid >= off) mx = fmax(mx, up);
-                }
-                double before = __shfl_up_sync(0xffffffffu, mx, 1);
-                before = tid ? fmax(before, (double)m0) : (double)m0;
-#pragma unroll
-                for (int e = 0; e < 2; ++e) {
-                    const uint32_t r = 2 * tid + e;
-                    bs[r] = b[e];
-                    ig[r] = iv[e];
-                    mr[r] = (float)(b[e] + fmax(before, x[e]));
-                    rowf[r] = expf((float)((double)m0 + b[e] - (double)mr[r]));
-                }
+                block_gates(a, h, tid, m0, zi, zf, bg);
             }
             __syncthreads();
             if (tid < C) {
-                colf[tid] = tid < n ? expf((float)(bs[n - 1] - bs[tid] + (double)ig[tid] - (double)mr[n - 1])) : 0.0f;
-                if (tid == 0) keep_s = rowf[n - 1];
+                colf[tid] = tid < n ? expf((float)(bg.rowd(n - 1) + bg.cold(tid))) : 0.0f;
+                if (tid == 0) keep_s = bg.rowf[n - 1];
             }
-            m0 = mr[n - 1];
+            m0 = bg.m[n - 1];
         } else if (tid < C) {
-            rowf[tid] = pw[tid + 1];
+            bg.rowf[tid] = pw[tid + 1];
             colf[tid] = tid < n ? pw[n - 1 - tid] : 0.0f;
             if (tid == 0) keep_s = pw[n];
         }
@@ -438,7 +394,7 @@ recurrence_chunk_kernel(QbRecurrence a, uint32_t dimr) {
                 for (int j = 0; j < 4; ++j) {
                     const uint32_t ri = ty * 4 + i, cj = tx + 16 * j;
                     if constexpr (GATED)
-                        pm[ri * PP + cj] = cj <= ri ? acc[i][j] * expf((float)(bs[ri] - bs[cj] + (double)ig[cj] - (double)mr[ri])) : 0.0f;
+                        pm[ri * PP + cj] = cj <= ri ? acc[i][j] * expf((float)(bg.rowd(ri) + bg.cold(cj))) : 0.0f;
                     else
                         pm[ri * PP + cj] = cj <= ri ? acc[i][j] * pw[ri - cj] : 0.0f;
                 }
@@ -465,7 +421,7 @@ recurrence_chunk_kernel(QbRecurrence a, uint32_t dimr) {
 #pragma unroll
             for (int k = 0; k < 2; ++k)
 #pragma unroll
-                for (int i = 0; i < 4; ++i) o[k][i] *= rowf[r + 32 * k];
+                for (int i = 0; i < 4; ++i) o[k][i] *= bg.rowf[r + 32 * k];
             for (uint32_t j = 0; j < C; j += 4) {
                 float4 vv[4];
 #pragma unroll
@@ -492,13 +448,13 @@ recurrence_chunk_kernel(QbRecurrence a, uint32_t dimr) {
             float nq = 0.0f, ps = 0.0f;
             for (uint32_t d = p; d < dimr; d += 4) nq = fmaf(qs[r * dp + d], nst[d], nq);
             for (uint32_t j = p; j < C; j += 4) ps += pm[r * PP + j];
-            nq = fmaf(nq, rowf[r], ps);
+            nq = fmaf(nq, bg.rowf[r], ps);
             nq += __shfl_xor_sync(0xffffffffu, nq, 1);
             nq += __shfl_xor_sync(0xffffffffu, nq, 2);
             if (p == 0 && r < n) {
                 float *aux = a.row_aux + (((size_t)s * a.R + r0 + r) * a.H + h) * 2;
                 aux[0] = nq;
-                aux[1] = mr[r];
+                aux[1] = bg.m[r];
             }
         }
         __syncthreads();
@@ -595,34 +551,38 @@ int launch_step(qb_ctx *ctx, const QbRecurrence &a) {
         const uint32_t ni = (a.dim + RT / (vc / 4) - 1) / (RT / (vc / 4)), split = (a.vdim + vc - 1) / vc;
         const size_t smem = ((size_t)2 * a.dim + (RT / 32) * vc) * sizeof(float);
         if (split <= 8 && ni <= 16) {
-            if (ni <= 2) return launch_cluster(ctx, recurrence_decode_kernel<T, 2, GATED>, a, vc, smem, "recurrence_decode_kernel");
-            if (ni <= 4) return launch_cluster(ctx, recurrence_decode_kernel<T, 4, GATED>, a, vc, smem, "recurrence_decode_kernel");
-            if (ni <= 8) return launch_cluster(ctx, recurrence_decode_kernel<T, 8, GATED>, a, vc, smem, "recurrence_decode_kernel");
-            return launch_cluster(ctx, recurrence_decode_kernel<T, 16, GATED>, a, vc, smem, "recurrence_decode_kernel");
+            if (ni <= 2) return launch_cluster(ctx, recurrence_decode_kernel<T, 2, GATED>, a, vc, smem, GATED ? "gated_recurrence_decode_kernel" : "recurrence_decode_kernel");
+            if (ni <= 4) return launch_cluster(ctx, recurrence_decode_kernel<T, 4, GATED>, a, vc, smem, GATED ? "gated_recurrence_decode_kernel" : "recurrence_decode_kernel");
+            if (ni <= 8) return launch_cluster(ctx, recurrence_decode_kernel<T, 8, GATED>, a, vc, smem, GATED ? "gated_recurrence_decode_kernel" : "recurrence_decode_kernel");
+            return launch_cluster(ctx, recurrence_decode_kernel<T, 16, GATED>, a, vc, smem, GATED ? "gated_recurrence_decode_kernel" : "recurrence_decode_kernel");
         }
     }
     uint32_t vc = VCH;
     while ((a.vdim + vc - 1) / vc > 8) vc += VCH;
     return launch_cluster(ctx, recurrence_step_kernel<T, GATED>, a, vc, ((size_t)a.dim * vc + 3 * a.dim + a.rot.dims + (RT / 32) * vc) * sizeof(float),
-                          "recurrence_step_kernel");
+                          GATED ? "gated_recurrence_step_kernel" : "recurrence_step_kernel");
 }
 
 template <bool GATED>
 int launch(qb_ctx *ctx, const QbRecurrence &a) {
     const uint32_t dimr = (a.dim + 3) & ~3u;
     const size_t smem = ((size_t)2 * C * (dimr + 4) + C * VCH + (size_t)dimr * VCH + C * (C + 4) + C + 4 + dimr) * sizeof(float);
-    if (a.R < 16 || smem > 220 * 1024) return a.out.f32 ? launch_step<float, GATED>(ctx, a) : launch_step<__nv_bfloat16, GATED>(ctx, a);
+    if (a.R < 16 || (smem > 220 * 1024 && !qb_recurrence_mma_supports(a))) return a.out.f32 ? launch_step<float, GATED>(ctx, a) : launch_step<__nv_bfloat16, GATED>(ctx, a);
     if (a.S > 1 || a.rot.dims) {
         QB_CUDA(qb_launch_pdl(ctx->stream, recurrence_rotate_kernel, dim3(a.ns * a.R), dim3(RT), (size_t)(a.rot.dims * sizeof(float)), a));
-        QB_LAUNCHED(ctx, "recurrence_rotate_kernel");
+        QB_LAUNCHED(ctx, GATED ? "gated_recurrence_rotate_kernel" : "recurrence_rotate_kernel");
     }
-    QB_CUDA(cudaFuncSetAttribute(recurrence_chunk_kernel<GATED>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-    QB_CUDA(qb_launch_pdl(ctx->stream, recurrence_chunk_kernel<GATED>, dim3(qb_recurrence_slices(a.vdim), a.H, a.ns), dim3(RT), smem, a, dimr));
-    QB_LAUNCHED(ctx, "recurrence_chunk_kernel");
+    if (qb_recurrence_mma_supports(a)) {
+        QB_TRY(qb_launch_recurrence_mma(ctx, a));
+    } else {
+        QB_CUDA(cudaFuncSetAttribute(recurrence_chunk_kernel<GATED>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+        QB_CUDA(qb_launch_pdl(ctx->stream, recurrence_chunk_kernel<GATED>, dim3(qb_recurrence_slices(a.vdim), a.H, a.ns), dim3(RT), smem, a, dimr));
+        QB_LAUNCHED(ctx, GATED ? "gated_recurrence_chunk_kernel" : "recurrence_chunk_kernel");
+    }
     const dim3 grid((a.ns * a.R * a.H + RT / 32 - 1) / (RT / 32));
     if (a.out.f32) QB_CUDA(qb_launch_pdl(ctx->stream, recurrence_gate_kernel<float, GATED>, grid, dim3(RT), (size_t)0, a));
     else QB_CUDA(qb_launch_pdl(ctx->stream, recurrence_gate_kernel<__nv_bfloat16, GATED>, grid, dim3(RT), (size_t)0, a));
-    QB_LAUNCHED(ctx, "recurrence_gate_kernel");
+    QB_LAUNCHED(ctx, GATED ? "gated_recurrence_gate_kernel" : "recurrence_gate_kernel");
     return QB_OK;
 }
 

@@ -70,7 +70,27 @@ shared_kv_prepare_kernel(QbSharedKv a) {
     }
 }
 
-// A warp per (row, head): the spans' weights, the sink, the gate.
+// What the merge of (row m, head h) reads: its spans, how many of them are visible, the sink's share and the gate.
+struct Merge { const float *ml, *acc; uint32_t n; float mx, factor; };
+__device__ __forceinline__ Merge merge_of(const QbSharedKv &a, uint32_t m, uint32_t h, uint32_t n_splits, uint32_t lane) {
+    const QbLatent &L = a.at;
+    const uint32_t s = m / L.R, r = m % L.R, hg = L.heads_per_group(), base = (uint32_t)L.seq_pos[s];
+    const size_t q = (((size_t)s * L.groups + h / hg) * L.R + r) * hg + h % hg;
+    const float g = qb_sum8(a.proj, (size_t)m * a.stride + (size_t)(L.H + L.groups) * L.rank + h, a.S, (size_t)L.ns * L.R * a.stride);
+    Merge o;
+    o.ml = L.part_ml + q * n_splits * 2;
+    o.acc = L.part_acc + q * n_splits * L.rank;
+    o.n = min((base + r) / qb_latent_span(base + L.R, L.max_splits) + 1, n_splits);
+    o.mx = 0.0f;                                              // the sink's score
+    for (uint32_t i = lane; i < o.n; i += 32) o.mx = fmaxf(o.mx, o.ml[2 * i]);
+    o.mx = warp_max(o.mx);
+    float den = 0.0f;
+    for (uint32_t i = lane; i < o.n; i += 32) den += o.ml[2 * i + 1] * expf(o.ml[2 * i] - o.mx);
+    o.factor = qb_sigmoid(g) / (warp_sum(den) + expf(-o.mx));
+    return o;
+}
+
+// Few spans: a warp per (row, head).
 template <typename T>
 __global__ void __launch_bounds__(ST)
 shared_kv_merge_kernel(QbSharedKv a, uint32_t n_splits) {
@@ -78,39 +98,71 @@ shared_kv_merge_kernel(QbSharedKv a, uint32_t n_splits) {
     const QbLatent &L = a.at;
     const uint32_t t = blockIdx.x * (ST / 32) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
     if (t >= L.ns * L.R * L.H) return;
-    const uint32_t m = t / L.H, h = t % L.H, s = m / L.R, r = m % L.R, hg = L.heads_per_group();
-    const uint32_t base = (uint32_t)L.seq_pos[s], n = min((base + r) / qb_latent_span(base + L.R, L.max_splits) + 1, n_splits);
-    const size_t q = (((size_t)s * L.groups + h / hg) * L.R + r) * hg + h % hg;
-    const float *ml = L.part_ml + q * n_splits * 2, *acc = L.part_acc + q * n_splits * L.rank;
-    float mx = 0.0f;                                          // the sink's score
-    for (uint32_t i = lane; i < n; i += 32) mx = fmaxf(mx, ml[2 * i]);
-    mx = warp_max(mx);
-    float den = 0.0f;
-    for (uint32_t i = lane; i < n; i += 32) den += ml[2 * i + 1] * expf(ml[2 * i] - mx);
-    den = warp_sum(den) + expf(-mx);
-    const float gate = qb_sigmoid(qb_sum8(a.proj, (size_t)m * a.stride + (size_t)(L.H + L.groups) * L.rank + h, a.S, (size_t)L.ns * L.R * a.stride)) / den;
+    const uint32_t m = t / L.H, h = t % L.H;
+    const Merge o = merge_of(a, m, h, n_splits, lane);
     T *out = (T *)L.out.p + (size_t)m * L.out.ld + (size_t)h * L.rank;
     for (uint32_t c = lane; c < L.rank; c += 32) {
         float v = 0.0f;
-#pragma unroll 8
-        for (uint32_t i = 0; i < n; ++i) v = fmaf(expf(ml[2 * i] - mx), acc[(size_t)i * L.rank + c], v);
-        out[c] = qb_cast<T>(v * gate);
+#pragma unroll 4
+        for (uint32_t i = 0; i < o.n; ++i) v = fmaf(expf(o.ml[2 * i] - o.mx), o.acc[(size_t)i * L.rank + c], v);
+        out[c] = qb_cast<T>(v * o.factor);
+    }
+}
+// Many spans: a CTA per (row, head), its warps take spans by turns, 128 columns at a time.
+template <typename T>
+__global__ void __launch_bounds__(ST)
+shared_kv_merge_wide_kernel(QbSharedKv a, uint32_t n_splits) {
+    QB_PDL_ENTER();
+    __shared__ float part[ST / 32][128];
+    const QbLatent &L = a.at;
+    const uint32_t m = blockIdx.x / L.H, h = blockIdx.x % L.H, w = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const Merge o = merge_of(a, m, h, n_splits, lane);
+    T *out = (T *)L.out.p + (size_t)m * L.out.ld + (size_t)h * L.rank;
+    for (uint32_t c0 = 0; c0 < L.rank; c0 += 128) {
+        float v[4] = {};
+#pragma unroll 4
+        for (uint32_t i = w; i < o.n; i += ST / 32) {
+            const float e = expf(o.ml[2 * i] - o.mx), *acc = o.acc + (size_t)i * L.rank + c0 + lane;
+#pragma unroll
+            for (int j = 0; j < 4; ++j)
+                if (c0 + lane + 32 * j < L.rank) v[j] = fmaf(e, acc[32 * j], v[j]);
+        }
+#pragma unroll
+        for (int j = 0; j < 4; ++j) part[w][lane + 32 * j] = v[j];
+        __syncthreads();
+        const uint32_t c = threadIdx.x;
+        if (c < 128 && c0 + c < L.rank) {
+            float t = 0.0f;
+#pragma unroll
+            for (int i = 0; i < ST / 32; ++i) t += part[i][c];
+            out[c0 + c] = qb_cast<T>(t * o.factor);
+        }
+        __syncthreads();
     }
 }
 
+template <typename T>
+int launch_merge(qb_ctx *ctx, const QbSharedKv &a, uint32_t n_splits) {
+    const uint32_t n = a.at.ns * a.at.R * a.at.H;
+    if (n_splits > 4) QB_CUDA(qb_launch_pdl(ctx->stream, shared_kv_merge_wide_kernel<T>, dim3(n), dim3(ST), (size_t)0, a, n_splits));
+    else QB_CUDA(qb_launch_pdl(ctx->stream, shared_kv_merge_kernel<T>, dim3((n + ST / 32 - 1) / (ST / 32)), dim3(ST), (size_t)0, a, n_splits));
+    QB_LAUNCHED(ctx, "shared_kv_merge_kernel");
+    return QB_OK;
+}
+
 // Queries a span kernel's CTA takes at most (what fills the GPU is counted in these).
-constexpr uint32_t SPAN_QUERIES = 48, MAX_SPANS = 64;
+constexpr uint32_t SPAN_QUERIES = 48, MAX_SPANS = 64, CTAS_PER_SM = 6;
 
 }  // namespace
 
-// Spans per sequence that fill the GPU with a few CTAs per SM.
+// Spans per sequence that fill the GPU about twice over with the CTAs that small tiles leave room for on an SM.
 uint32_t qb_shared_kv_max_splits(const QbLatent &a, uint32_t ns, uint32_t R, uint32_t sms) {
     const uint64_t ctas = (uint64_t)ns * a.groups * ((R * a.heads_per_group() + SPAN_QUERIES - 1) / SPAN_QUERIES);
-    return (uint32_t)std::max<uint64_t>(1, std::min<uint64_t>(MAX_SPANS, 3ull * sms / ctas));
+    return (uint32_t)std::max<uint64_t>(1, std::min<uint64_t>(MAX_SPANS, (uint64_t)CTAS_PER_SM * sms / ctas));
 }
 size_t qb_shared_kv_part_floats(const QbLatent &a, uint32_t rows_cap, uint32_t n_seqs, uint32_t sms) {
     // (queries x spans): at most one span per query, or CTAs x queries of a CTA
-    const size_t many = (size_t)std::max(rows_cap, n_seqs) * a.H, few = (size_t)3 * sms * SPAN_QUERIES;
+    const size_t many = (size_t)std::max(rows_cap, n_seqs) * a.H, few = (size_t)CTAS_PER_SM * sms * SPAN_QUERIES;
     return std::max(many, few) * a.rank;
 }
 
@@ -131,9 +183,5 @@ int qb_launch_shared_kv(qb_ctx *ctx, const QbSharedKv &args) {
     const uint32_t n_splits = std::min(L.max_splits, (L.max_pos + 63) / 64);
     if (qb_latent_tc_supports(L)) QB_TRY(qb_launch_latent_split_tc(ctx, L, n_splits));
     else QB_TRY(qb_launch_latent_split_simt(ctx, L, n_splits));
-    const dim3 mgrid((rows * L.H + ST / 32 - 1) / (ST / 32));
-    if (L.f32) QB_CUDA(qb_launch_pdl(ctx->stream, shared_kv_merge_kernel<float>, mgrid, dim3(ST), (size_t)0, a, n_splits));
-    else QB_CUDA(qb_launch_pdl(ctx->stream, shared_kv_merge_kernel<__nv_bfloat16>, mgrid, dim3(ST), (size_t)0, a, n_splits));
-    QB_LAUNCHED(ctx, "shared_kv_merge_kernel");
-    return QB_OK;
+    return L.f32 ? launch_merge<float>(ctx, a, n_splits) : launch_merge<__nv_bfloat16>(ctx, a, n_splits);
 }

@@ -2,10 +2,20 @@
 
 Test infrastructure only: it shares no code with the product path.  `dt` is the number type of everything (float64 unless
 a test asks for float32).  Weights are a dict {tensor name: array}, the configuration the parsed config.json.
+`rnd` is applied to what enters a matrix product from the right of a weight (identity unless a test asks what rounding those
+operands does to a row).
 """
 import numpy as np
 
 from kezilix_oracle import bf16_round, rms, rms_norm, silu, write_model  # noqa: F401  (plain helpers, shared between the oracles)
+
+
+def exact(a):
+    return a
+
+
+def to_bf16(a):
+    return bf16_round(a.astype(np.float32)).astype(a.dtype)
 
 
 def sigmoid(z):
@@ -35,14 +45,15 @@ def rotate(x, pos, rot):
     return np.concatenate([u * np.cos(a) - v * np.sin(a), v * np.cos(a) + u * np.sin(a), x[..., n:]], -1)
 
 
-def attention(h, w, mx, eps, pos=None):
+def attention(h, w, mx, eps, pos=None, rnd=exact):
     """Grouped-query attention whose values are the raw key projections, with a zero-score sink and one gate per head."""
     dt = h.dtype.type
     T, H, G, d = len(h), mx["heads"], mx["kv_heads"], mx["dim"]
     pos = np.arange(T) if pos is None else pos
     raw = (h @ w["k"].T).reshape(T, G, d)
-    q = rotate(rms_norm((h @ w["q"].T).reshape(T, H, d), w["q.norm"], eps), pos, mx["rot"])
-    k = rotate(rms_norm(raw, w["k.norm"], eps), pos, mx["rot"])
+    q = rnd(rotate(rms_norm((h @ w["q"].T).reshape(T, H, d), w["q.norm"], eps), pos, mx["rot"]))
+    k = rnd(rotate(rms_norm(raw, w["k.norm"], eps), pos, mx["rot"]))
+    raw = rnd(raw)
     o = np.zeros((T, H, d), h.dtype)
     for n in range(H):
         g = n // (H // G)
@@ -52,7 +63,7 @@ def attention(h, w, mx, eps, pos=None):
         e = np.exp(s - m[:, None])
         o[:, n] = (e / (e.sum(-1) + np.exp(-m))[:, None]) @ raw[:, g]
     o = o * sigmoid(h @ w["g"].T)[:, :, None]
-    return o.reshape(T, H * d) @ w["o"].T
+    return rnd(o.reshape(T, H * d)) @ w["o"].T
 
 
 def lightning_core(q, k, v, decay):
@@ -67,12 +78,12 @@ def lightning_core(q, k, v, decay):
     return o
 
 
-def lightning(h, w, mx, eps, pos=None):
+def lightning(h, w, mx, eps, pos=None, rnd=exact):
     T, H, d, vd = len(h), mx["heads"], mx["dim"], mx["vdim"]
     q, k = (silu(h @ w[n].T).reshape(T, H, d) for n in ("q", "k"))
     v = silu(h @ w["v"].T).reshape(T, H, vd)
     o = lightning_core(q, k, v, mx["decay"]).reshape(T, H * vd)
-    return (rms_norm(o, w["norm"], eps) * sigmoid(h @ w["g"].T)) @ w["o"].T
+    return rnd(rms_norm(o, w["norm"], eps) * sigmoid(h @ w["g"].T)) @ w["o"].T
 
 
 def log_sigmoid(z):
@@ -104,7 +115,7 @@ def mlstm_gates(h, w, cap):
     return soft_cap(h @ w["i"].T + w["i.b"], cap), log_sigmoid(soft_cap(h @ w["f"].T + w["f.b"], cap))
 
 
-def mlstm(h, w, mx, eps, pos=None):
+def mlstm(h, w, mx, eps, pos=None, rnd=exact):
     dt = h.dtype.type
     T, H, d, vd = len(h), mx["heads"], mx["dim"], mx["vdim"]
     q = (h @ w["q"].T).reshape(T, H, d) * dt(d ** -0.5)
@@ -112,14 +123,14 @@ def mlstm(h, w, mx, eps, pos=None):
     v = (h @ w["v"].T).reshape(T, H, vd)
     i, f = mlstm_gates(h, w, dt(mx["gate_cap"]))
     o = rms(mlstm_core(q, k, v, i, f), eps).reshape(T, H * vd)
-    return (o * w["norm"] * sigmoid(h @ w["g"].T)) @ w["o"].T
+    return rnd(o * w["norm"] * sigmoid(h @ w["g"].T)) @ w["o"].T
 
 
 MIXERS = {"attention": attention, "lightning": lightning, "mlstm": mlstm}
 
 
-def dense_ff(h, w):
-    return (silu(h @ w["gate"].T) * (h @ w["up"].T)) @ w["down"].T
+def dense_ff(h, w, rnd=exact):
+    return rnd(silu(h @ w["gate"].T) * (h @ w["up"].T)) @ w["down"].T
 
 
 def weights_of(cfg, i):
@@ -129,7 +140,7 @@ def weights_of(cfg, i):
     return i
 
 
-def forward(cfg, weights, tokens, dt=np.float64, trace=None):
+def forward(cfg, weights, tokens, dt=np.float64, trace=None, rnd=exact):
     """Logits [T][vocab] of one sequence; trace (a list) receives the residual stream after every layer."""
     W = {k: np.asarray(v, dt) for k, v in weights.items()}
     eps = cfg["norm"]["eps"]
@@ -137,12 +148,12 @@ def forward(cfg, weights, tokens, dt=np.float64, trace=None):
     x = W["embed"][np.asarray(tokens)] * dt(cfg["embedding"]["scale"])
     for i, L in enumerate(cfg["layers"]):
         p = "l%d." % weights_of(cfg, i)
-        x = x + layer_norm(MIXERS[L["type"]](x, sub(p + "mix."), L["mixer"], eps), W[p + "norm1"], eps) * W[p + "ls1"]
+        x = x + layer_norm(MIXERS[L["type"]](rnd(x), sub(p + "mix."), L["mixer"], eps, rnd=rnd), W[p + "norm1"], eps) * W[p + "ls1"]
         if L.get("mlp"):
-            x = x + layer_norm(dense_ff(x, sub(p + "mlp.")), W[p + "norm2"], eps) * W[p + "ls2"]
+            x = x + layer_norm(dense_ff(rnd(x), sub(p + "mlp."), rnd), W[p + "norm2"], eps) * W[p + "ls2"]
         if trace is not None:
             trace.append(x.copy())
-    return layer_norm(x, W["final.norm"], eps) @ W["head"].T
+    return rnd(layer_norm(x, W["final.norm"], eps)) @ W["head"].T
 
 
 def tensor_shapes(cfg):

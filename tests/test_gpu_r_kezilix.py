@@ -17,9 +17,10 @@ pytestmark = pytest.mark.gpu
 
 ROOT = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
 sys.path.insert(0, os.path.join(ROOT, "oracle"))
+sys.path.insert(0, os.path.join(ROOT, "tests"))
 import kezilix_oracle as K  # noqa: E402
+from layered_case import TOL, Case, close_to, in_portions  # noqa: E402
 
-TOL = {"float32": 3e-5, "bfloat16": 4e-2}
 YARN = {"factor": 6.0, "original": 256, "fast": 24.0, "slow": 2.0}
 
 
@@ -44,66 +45,16 @@ MIXED = config([lat(), ret(), ret(heads=2, dim=40, vdim=24, rot=40, decay=(0.99,
                loop={"start": 1, "stop": 4, "times": 2})
 
 
-class Case:
-    """A configuration with seeded weights, loaded from files in one or both number formats."""
-
-    def __init__(self, qb, ctx, tmp, cfg, seed=1, edit=None):
-        self.qb, self.ctx, self.cfg = qb, ctx, cfg
-        self.W = K.random_weights(cfg, seed)
-        if edit:
-            edit(self.W)
-        self.dir = str(tmp)
-        K.write_model(self.dir, cfg, self.W)
-        self.models = {}
-        self.rng = np.random.default_rng(seed + 100)
-
-    def model(self, dtype):
-        if dtype not in self.models:
-            self.models[dtype] = self.qb.Model.load(self.ctx, self.dir, dtype)
-        return self.models[dtype]
-
-    def batch(self, dtype, n_seqs=1, max_ctx=512, **kw):
-        return self.qb.Batch(self.model(dtype), n_seqs, max_ctx, 0, **kw)
-
-    def tokens(self, n):
-        return self.rng.integers(0, self.cfg["vocab"], n).tolist()
-
-    def want(self, tokens, trace=None):
-        return K.forward(self.cfg, self.W, tokens, np.float64, trace)
-
-    def close(self):
-        for m in self.models.values():
-            m.close()
-
-
 @pytest.fixture
 def make(qb, ctx, tmp_path):
     made = []
 
     def f(cfg, **kw):
-        made.append(Case(qb, ctx, tmp_path / ("m%d" % len(made)), cfg, **kw))
+        made.append(Case(K, qb, ctx, tmp_path / ("m%d" % len(made)), cfg, **kw))
         return made[-1]
     yield f
     for c in made:
         c.close()
-
-
-def close_to(got, want, dtype, what=""):
-    """Root-mean-square difference per row relative to the rms of the whole expected array."""
-    assert np.isfinite(got).all(), what
-    e = np.sqrt(((got - want) ** 2).mean(-1)) / np.sqrt((want ** 2).mean())
-    assert e.max() < TOL[dtype], "%s: row %d differs by %.3g" % (what, int(e.argmax()), e.max())
-
-
-def in_portions(b, seq, tokens, size):
-    """Logits at every position, the tokens cut into portions of `size` (a number, or a list that repeats)."""
-    out, at, i = [], 0, 0
-    sizes = [size] if isinstance(size, int) else size
-    while at < len(tokens):
-        n = min(sizes[i % len(sizes)], len(tokens) - at)
-        out.append(b.score(seq, tokens[at:at + n], range(n)))
-        at, i = at + n, i + 1
-    return np.concatenate(out)
 
 
 # ---- products ----------------------------------------------------------------------------------------------------------
@@ -394,19 +345,12 @@ def test_state_reaches_far_back(make):
 
 
 # ---- generation through the scheduler -------------------------------------------------------------------------------------------
-def greedy_oracle(c, prompt, n):
-    seq = list(prompt)
-    for _ in range(n):
-        seq.append(int(c.want(seq)[-1].argmax()))
-    return seq[len(prompt):]
-
-
 @pytest.mark.parametrize("loop", ["run", "run_compact", "prefix_cache"])
 def test_greedy_generation_through_the_scheduler(qb, make, loop):
     c = make(MIXED)
     shared = c.tokens(32)
     prompts = [shared + c.tokens(9), c.tokens(3), shared + c.tokens(20), c.tokens(70), c.tokens(1)]
-    want = [greedy_oracle(c, p, 12) for p in prompts]
+    want = [c.greedy(p, 12) for p in prompts]
     reqs = [qb.serve.Request(i, p, 12, arrival_step=6 * i) for i, p in enumerate(prompts)]
     if loop == "run":
         b = c.batch("float32", n_seqs=2, max_ctx=160)
@@ -433,10 +377,10 @@ def test_sampled_generation(qb, make):
         qb.serve.run_compact(b, reqs, speculative=False, sampling=sampling, rng_of=lambda r: random.Random(7 + r.rid))
         b.close()
         return [r.tokens for r in reqs]
-    assert serve([0, 1, 2], 3, temp=0.8, top_k=1) == [greedy_oracle(c, p, 16) for p in prompts]
+    assert serve([0, 1, 2], 3, temp=0.8, top_k=1) == [c.greedy(p, 16) for p in prompts]
     together = serve([0, 1, 2], 3, temp=1.1, top_k=20, top_p=0.95)
     assert together == [serve([i], 1, temp=1.1, top_k=20, top_p=0.95)[0] for i in range(3)]
-    assert together != [greedy_oracle(c, p, 16) for p in prompts]
+    assert together != [c.greedy(p, 16) for p in prompts]
     pen = serve([0, 1, 2], 3, temp=0.01, presence=50.0)                       # a heavy presence penalty: no token twice
     assert all(len(set(p + t)) == len(set(p)) + len(t) for p, t in zip(prompts, pen))
 
@@ -492,4 +436,4 @@ def test_trace_replay_and_generate_programs(make, tmp_path):
     p = subprocess.run([os.path.join(ROOT, "bin", "generate"), "--model", c.dir, "--dtype", "float32", "--new-tokens", "8", "--slots", "2",
                         "--prompt", ",".join(map(str, a)), "--prompt", ",".join(map(str, d)), "--prompt", "5"], capture_output=True, text=True, timeout=300)
     assert p.returncode == 0, p.stderr[-500:]
-    assert [[int(t) for t in ln.split(",")] for ln in p.stdout.split()] == [greedy_oracle(c, q, 8) for q in (a, d, [5])]
+    assert [[int(t) for t in ln.split(",")] for ln in p.stdout.split()] == [c.greedy(q, 8) for q in (a, d, [5])]
