@@ -208,4 +208,7 @@ struct QbSharedKv {
 };
 uint32_t qb_shared_kv_max_splits(const QbLatent &a, uint32_t ns, uint32_t R, uint32_t sms);
 size_t qb_shared_kv_part_floats(const QbLatent &a, uint32_t rows_cap, uint32_t n_seqs, uint32_t sms);
+// Many prompt rows in one pass over the keys, up to the gated output (shared_kv_prefill_tc.cu): bfloat16, 16-key pages.
+bool qb_shared_kv_prefill_supports(const QbLatent &a, uint32_t sms);
+int qb_launch_shared_kv_prefill(qb_ctx *ctx, const QbSharedKv &a);
 int qb_launch_shared_kv(qb_ctx *ctx, const QbSharedKv &a);

@@ -9,7 +9,7 @@
 //
 // Three launches: shared_kv_prepare_kernel (norms, rotation, append), the spans over the cached vectors (the kernels of absorbed
 // latent attention with a group per key/value head: tcgen05 in bfloat16, fp32 arithmetic otherwise), shared_kv_merge_kernel
-// (spans, sink, gate).  Scores, weights and their sums are fp32.
+// (spans, sink, gate).  Many prompt rows in bfloat16: shared_kv_prefill_kernel instead of the last two.  Scores, weights and their sums are fp32.
 #include "layered.h"
 
 namespace {
@@ -180,6 +180,7 @@ int qb_launch_shared_kv(qb_ctx *ctx, const QbSharedKv &args) {
     if (L.f32) QB_CUDA(qb_launch_pdl(ctx->stream, shared_kv_prepare_kernel<float>, grid, dim3(ST), smem, a));
     else QB_CUDA(qb_launch_pdl(ctx->stream, shared_kv_prepare_kernel<__nv_bfloat16>, grid, dim3(ST), smem, a));
     QB_LAUNCHED(ctx, "shared_kv_prepare_kernel");
+    if (qb_shared_kv_prefill_supports(L, (uint32_t)ctx->sm_count)) return qb_launch_shared_kv_prefill(ctx, a);
     const uint32_t n_splits = std::min(L.max_splits, (L.max_pos + 63) / 64);
     if (qb_latent_tc_supports(L)) QB_TRY(qb_launch_latent_split_tc(ctx, L, n_splits));
     else QB_TRY(qb_launch_latent_split_simt(ctx, L, n_splits));

@@ -144,6 +144,20 @@ def test_decode_attention_shapes(make, heads, kv, dim, rot, n_seqs):
     b.close()
 
 
+@pytest.mark.parametrize("heads,kv,dim,rot", [(8, 2, 128, 32), (6, 2, 64, 64), (5, 1, 20, 12), (4, 4, 96, 8), (12, 3, 32, 4), (4, 1, 256, 64), (2, 2, 136, 40), (3, 1, 10, 2)])
+def test_prompt_attention_shapes(make, heads, kv, dim, rot):
+    """Prompt rows in tiles of 128 queries and 128 keys, cut at odd places: part of a tile, tiles across portions; one or two
+    buffers of keys, head sizes that are no multiples of 16 or 8; a raised scale lets the running maximum move."""
+    c = make(config([att(heads=heads, kv=kv, dim=dim, rot=rot, scale=5.0 / dim ** 0.5, ff=None)], eps=1e-3))
+    toks = c.tokens(700)
+    want = c.want(toks)
+    b = c.batch("bfloat16", max_ctx=704, page_order=1)
+    for size in (700, [301, 128, 1, 130]):
+        b.reset(0)
+        close_to(in_portions(b, 0, toks, size), want, "bfloat16", str(size), c.slack(toks))
+    b.close()
+
+
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
 @pytest.mark.parametrize("page", [8, 48])
 def test_other_page_sizes(make, page, dtype):
